@@ -74,17 +74,30 @@ __device__ __forceinline__ float activate(float z, int act)
     }
 }
 
-// out[t, f] = act(g) * u; gate and up fill the two halves of a row of gu or alternate along it
+// out[t, f] = act(g) * u; gate and up fill the two halves of a row of gu or alternate along it; rows of out are `ldo`
+// elements apart.  `bias` [2 F] in the row's order (may be null).  act = HFB_ACT_CLAMPED_GLU: g = min(g, limit), u =
+// clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + offset).
 template <typename T>
-__global__ void glu_kernel(const T *gu, T *out, int F, size_t total, int interleaved, int act)
+__global__ void glu_kernel(const T *gu, const void *bias, int bias_dt, T *out, size_t ldo, int F, size_t total, int interleaved, int act,
+                           float limit, float alpha, float offset)
 {
     pdl_entry();
     pdl_sync_small();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
         const size_t t = i / F;
         const int f = (int)(i % F);
-        const float g = to_f32(gu[t * 2 * F + (interleaved ? 2 * f : f)]), u = to_f32(gu[t * 2 * F + (interleaved ? 2 * f + 1 : F + f)]);
-        out[i] = from_f32<T>(activate(g, act) * u);
+        const int cg = interleaved ? 2 * f : f, cu = interleaved ? 2 * f + 1 : F + f;
+        float g = to_f32(gu[t * 2 * F + cg]), u = to_f32(gu[t * 2 * F + cu]);
+        if (bias) { g += load_any(bias, bias_dt, cg); u += load_any(bias, bias_dt, cu); }
+        float h;
+        if (act == HFB_ACT_CLAMPED_GLU) {
+            g = fminf(g, limit);
+            u = fminf(fmaxf(u, -limit), limit);
+            h = g / (1.0f + expf(-alpha * g)) * (u + offset);
+        } else {
+            h = activate(g, act) * u;
+        }
+        out[t * ldo + f] = from_f32<T>(h);
     }
 }
 
@@ -102,6 +115,15 @@ __global__ void scale_kernel(float *x, size_t total, float s)
     pdl_entry();
     pdl_sync_small();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) x[i] *= s;
+}
+
+__global__ void softcap_kernel(float *x, size_t total, float cap)
+{
+    pdl_entry();
+    pdl_sync_small();
+    const float inv = 1.0f / cap;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
+        x[i] = cap * tanhf(x[i] * inv);
 }
 
 static unsigned blocks_for(size_t total)
@@ -145,13 +167,15 @@ extern "C" int hfb_dyt_residual(const void *y, int y_dt, int splits, const void 
     return check_pdl_launch(g_launch_err, "dyt_residual");
 }
 
-extern "C" int hfb_glu(const void *gu, void *out, int dt, int T, int F, int interleaved, int act, hfb_stream s)
+extern "C" int hfb_glu(const void *gu, const void *bias, int bias_dt, void *out, int dt, int64_t ldo, int T, int F, int interleaved, int act,
+                       float limit, float alpha, float offset, hfb_stream s)
 {
     if (T <= 0) return HFB_OK;
-    if (!valid_dt(dt) || F <= 0 || act < 0 || act > ACT_NONE) return fail(HFB_EINVAL, "glu: bad arguments");
-    const size_t total = (size_t)T * F;
-    if (dt == HFB_F32) g_launch_err = launch_pdl(glu_kernel<float>, dim3(blocks_for(total)), dim3(256), 0, (cudaStream_t)s, (const float *)gu, (float *)out, F, total, interleaved, act);
-    else g_launch_err = launch_pdl(glu_kernel<__nv_bfloat16>, dim3(blocks_for(total)), dim3(256), 0, (cudaStream_t)s, (const __nv_bfloat16 *)gu, (__nv_bfloat16 *)out, F, total, interleaved, act);
+    if (!valid_dt(dt) || F <= 0 || act < 0 || act > HFB_ACT_CLAMPED_GLU || (bias && !valid_dt(bias_dt)) || (ldo && ldo < F))
+        return fail(HFB_EINVAL, "glu: bad arguments");
+    const size_t total = (size_t)T * F, row = ldo ? (size_t)ldo : (size_t)F;
+    if (dt == HFB_F32) g_launch_err = launch_pdl(glu_kernel<float>, dim3(blocks_for(total)), dim3(256), 0, (cudaStream_t)s, (const float *)gu, bias, bias_dt, (float *)out, row, F, total, interleaved, act, limit, alpha, offset);
+    else g_launch_err = launch_pdl(glu_kernel<__nv_bfloat16>, dim3(blocks_for(total)), dim3(256), 0, (cudaStream_t)s, (const __nv_bfloat16 *)gu, bias, bias_dt, (__nv_bfloat16 *)out, row, F, total, interleaved, act, limit, alpha, offset);
     return check_pdl_launch(g_launch_err, "glu");
 }
 
@@ -162,6 +186,15 @@ extern "C" int hfb_act(const void *x, void *out, int dt, int64_t total, int act,
     if (dt == HFB_F32) g_launch_err = launch_pdl(act_kernel<float>, dim3(blocks_for((size_t)total)), dim3(256), 0, (cudaStream_t)s, (const float *)x, (float *)out, (size_t)total, act);
     else g_launch_err = launch_pdl(act_kernel<__nv_bfloat16>, dim3(blocks_for((size_t)total)), dim3(256), 0, (cudaStream_t)s, (const __nv_bfloat16 *)x, (__nv_bfloat16 *)out, (size_t)total, act);
     return check_pdl_launch(g_launch_err, "act");
+}
+
+// x = cap * tanh(x / cap)
+extern "C" int hfb_softcap(float *x, int64_t total, float cap, hfb_stream s)
+{
+    if (total <= 0) return HFB_OK;
+    if (!x || !(cap > 0.f)) return fail(HFB_EINVAL, "softcap: the cap must be positive");
+    g_launch_err = launch_pdl(softcap_kernel, dim3(blocks_for((size_t)total)), dim3(256), 0, (cudaStream_t)s, x, (size_t)total, cap);
+    return check_pdl_launch(g_launch_err, "softcap");
 }
 
 extern "C" int hfb_scale(float *x, int64_t total, float scale, hfb_stream s)

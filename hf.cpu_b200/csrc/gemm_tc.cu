@@ -56,6 +56,9 @@ struct GemmParams {
     int mode;
     int act;                           // EPI_SWIGLU: the gate's activation (0 silu, else an HFB_ACT_* code);
                                        // EPI_STORE: 0 none, else the HFB_ACT_* code applied to sum + bias
+    // EPI_SWIGLU: elements between rows of out (0: N / 2), and the constants of HFB_ACT_CLAMPED_GLU
+    long long ldo;
+    float glu_limit, glu_alpha, glu_offset;
     float *partial;                    // [splits, M, N] when mode == EPI_PARTIAL
     // mode == EPI_ROPE_KV (pair kernel, tiles of whole heads): the output is the q|k|v row of a token; bias, rounding
     // to bfloat16, rotation of the query and key heads by the token's position, queries to q_out, keys and values to
@@ -101,6 +104,14 @@ __device__ __forceinline__ float epi_act(float z, int act)
     return z / (1.0f + expf(-z));
 }
 
+// A gated pair with both halves clamped: g = min(g, limit), u = clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + offset).
+__device__ __forceinline__ float epi_clamped_glu(const GemmParams &p, float g, float u)
+{
+    g = fminf(g, p.glu_limit);
+    u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
+    return __fdividef(g, 1.0f + __expf(-p.glu_alpha * g)) * (u + p.glu_offset);
+}
+
 // One chunk of 16 accumulator columns of one row: v[i] is element (xr, y0 + i) of X . Y^T.
 // `live` false: the same instructions, nothing stored (the few-token form runs its epilogue once this way while the
 // first weights are on their way, so that its code is in the instruction cache when the first tile is done: fetched
@@ -116,15 +127,17 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams &p, const uint32
         const int odd = lane & 1;
         const int in_chunk = min(16, p.M - y0);                                  // the same for the whole warp
         const int n_tok = (live && (xr | 1) < p.N) ? in_chunk : 0;
-        const size_t half_n = (size_t)(p.N >> 1), at = (size_t)y0 * half_n + (size_t)(xr >> 1);
+        const size_t half_n = p.ldo ? (size_t)p.ldo : (size_t)(p.N >> 1), at = (size_t)y0 * half_n + (size_t)(xr >> 1);
+        const float b = (p.bias && xr < p.N) ? load_any(p.bias, p.bias_dt, xr) : 0.f;
+        const bool clamped = p.act == HFB_ACT_CLAMPED_GLU;
 #pragma unroll
         for (int j = 0; j < 8; j++) {
             if (2 * j >= in_chunk) break;
-            const float first = __uint_as_float(v[2 * j]), second = __uint_as_float(v[2 * j + 1]);
+            const float first = __uint_as_float(v[2 * j]) + b, second = __uint_as_float(v[2 * j + 1]) + b;
             const float their_first = __shfl_xor_sync(0xffffffffu, first, 1);
             const float their_second = __shfl_xor_sync(0xffffffffu, second, 1);
             const float g = odd ? their_second : first, u = odd ? second : their_first;
-            const float h = epi_act(g, p.act) * u;
+            const float h = clamped ? epi_clamped_glu(p, g, u) : epi_act(g, p.act) * u;
             const int i = 2 * j + odd;
             if (i < n_tok) {
                 if (p.out_dt == HFB_BF16) ((__nv_bfloat16 *)p.out)[at + (size_t)i * half_n] = __float2bfloat16_rn(h);
@@ -179,14 +192,24 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams &p, const uint32
     } else if (p.mode == EPI_SWIGLU) {
         // columns alternate gate, up: 8 pairs -> 8 outputs of row xr, out is [M, N/2]
         if (xr < p.M && y0 < p.N) {
-            float h[8];
+            float h[8], f[16];
 #pragma unroll
-            for (int i = 0; i < 8; i++) {
-                float g = __uint_as_float(v[2 * i]), u = __uint_as_float(v[2 * i + 1]);
-                h[i] = epi_act(g, p.act) * u;
+            for (int i = 0; i < 16; i++) f[i] = __uint_as_float(v[i]);
+            if (p.bias) {
+#pragma unroll
+                for (int i = 0; i < 16; i++)
+                    if (y0 + i < p.N) f[i] += load_any(p.bias, p.bias_dt, y0 + i);
             }
-            size_t o = (size_t)xr * (p.N >> 1) + (y0 >> 1);
-            if (y0 + 16 <= p.N && (p.N & 15) == 0 && p.out_dt == HFB_BF16) {
+            if (p.act == HFB_ACT_CLAMPED_GLU) {
+#pragma unroll
+                for (int i = 0; i < 8; i++) h[i] = epi_clamped_glu(p, f[2 * i], f[2 * i + 1]);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; i++) h[i] = epi_act(f[2 * i], p.act) * f[2 * i + 1];
+            }
+            const size_t ldo = p.ldo ? (size_t)p.ldo : (size_t)(p.N >> 1);
+            size_t o = (size_t)xr * ldo + (y0 >> 1);
+            if (y0 + 16 <= p.N && (ldo & 7) == 0 && p.out_dt == HFB_BF16) {
                 __nv_bfloat162 hh[4];
 #pragma unroll
                 for (int i = 0; i < 4; i++) hh[i] = __floats2bfloat162_rn(h[2 * i], h[2 * i + 1]);
@@ -1091,18 +1114,23 @@ extern "C" int hfb_linear_tc_swiglu(const void *a, const void *w, void *out, int
     return launch_bn(bn, mx, my, p, (cudaStream_t)s);
 }
 
-// The gated form with another activation of the gate than silu (an HFB_ACT_* code).
-extern "C" int hfb_linear_tc_glu(const void *a, const void *w, void *out, int out_dt, int M, int N, int K, int act, hfb_stream s)
+// The gated form with another activation of the gate than silu (an HFB_ACT_* code), a bias [N] in the rows' order
+// (may be null), output rows `ldo` elements apart (0: N / 2), and for HFB_ACT_CLAMPED_GLU its three constants.
+extern "C" int hfb_linear_tc_glu(const void *a, const void *w, const void *bias, int bias_dt, void *out, int out_dt, int64_t ldo, int M,
+                                 int N, int K, int act, float limit, float alpha, float offset, hfb_stream s)
 {
     if (M <= 0 || N <= 0) return HFB_OK;
     int rc = check_tc_args("linear_tc_glu", a, w, out, M, N, K);
     if (rc != HFB_OK) return rc;
-    if ((N & 1) || !valid_dt(out_dt) || act < 0 || act >= HFB_ACT_NONE) return fail(HFB_EINVAL, "linear_tc_glu: bad arguments");
+    if ((N & 1) || !valid_dt(out_dt) || act < 0 || (act >= HFB_ACT_NONE && act != HFB_ACT_CLAMPED_GLU) || (bias && !valid_dt(bias_dt)) ||
+        (ldo && ldo < N / 2))
+        return fail(HFB_EINVAL, "linear_tc_glu: bad arguments");
     GemmParams p{};
     CUtensorMap mx, my;
     int bn;
     if ((rc = plan_and_maps(a, w, M, N, K, p, bn, mx, my)) != HFB_OK) return rc;
-    p.out = out; p.out_dt = out_dt; p.bias = nullptr; p.mode = EPI_SWIGLU; p.act = act;
+    p.out = out; p.out_dt = out_dt; p.bias = bias; p.bias_dt = bias_dt; p.mode = EPI_SWIGLU; p.act = act;
+    p.ldo = ldo; p.glu_limit = limit; p.glu_alpha = alpha; p.glu_offset = offset;
     return launch_bn(bn, mx, my, p, (cudaStream_t)s);
 }
 

@@ -66,7 +66,8 @@ int hfb_linear_tc_swiglu(const void *a, const void *w, void *out, int out_dt, in
 
 /* The gated product with another activation of the gate (HFB_ACT_* code), and out = act(a . w^T) with the activation in
  * the epilogue (act other than silu; K is never split). */
-int hfb_linear_tc_glu(const void *a, const void *w, void *out, int out_dt, int M, int N, int K, int act, hfb_stream s);
+int hfb_linear_tc_glu(const void *a, const void *w, const void *bias, int bias_dt, void *out, int out_dt, int64_t ldo, int M, int N, int K,
+                      int act, float limit, float alpha, float offset, hfb_stream s);
 int hfb_linear_tc_act(const void *a, const void *w, void *out, int out_dt, int M, int N, int K, int act, hfb_stream s);
 
 /* q|k|v of 256 tokens and more with the rest of the step in the product's epilogue: bias, rounding to bfloat16,
@@ -183,12 +184,17 @@ void hfb_set_launch_overlap(int on);
 int hfb_swiglu(const void *gu, void *out, int dt, int T, int F, int interleaved, hfb_stream s);
 
 /* Activations: codes for hfb_glu / hfb_act / the expert products. */
-enum { HFB_ACT_SILU = 0, HFB_ACT_RELU = 1, HFB_ACT_GELU_TANH = 2, HFB_ACT_RELU2 = 3, HFB_ACT_NONE = 4 };
+enum { HFB_ACT_SILU = 0, HFB_ACT_RELU = 1, HFB_ACT_GELU_TANH = 2, HFB_ACT_RELU2 = 3, HFB_ACT_NONE = 4,
+       /* a gated pair only: g = min(g, limit), u = clamp(u, -limit, limit), g * sigmoid(alpha g) * (u + offset) */
+       HFB_ACT_CLAMPED_GLU = 5 };
 /* added to the activation of hfb_moe_gemm: rows of w alternate gate, up, and out [.., N / 2] = act(gate) * up */
 enum { HFB_ACT_GLU = 256 };
 
 /* out[t, f] = act(g) * u, gate and up laid out as for hfb_swiglu */
-int hfb_glu(const void *gu, void *out, int dt, int T, int F, int interleaved, int act, hfb_stream s);
+int hfb_glu(const void *gu, const void *bias, int bias_dt, void *out, int dt, int64_t ldo, int T, int F, int interleaved, int act,
+            float limit, float alpha, float offset, hfb_stream s);
+/* x = cap * tanh(x / cap), float32 */
+int hfb_softcap(float *x, int64_t total, float cap, hfb_stream s);
 
 /* out[i] = act(x[i]) (in place when out == x) */
 int hfb_act(const void *x, void *out, int dt, int64_t total, int act, hfb_stream s);
@@ -316,6 +322,48 @@ int hfb_linear_scan(const float *q, int q_stride, const float *k, int k_stride, 
                     int n_slots, int S, float *o, int o_stride, int H, int Hq, int d, int dv, hfb_stream s);
 int hfb_gate_norm(const float *o, const void *w, int w_dt, float eps, const float *g, int g_splits, int g_stride,
                   int g_col0, int gate, void *out, int out_dt, int T, int H, int dv, hfb_stream s);
+
+/* conv_carry: the carried inputs [taps - 1][C] of a causal convolution after a step (channel c = column x_col0 + c of rows
+ * x_stride floats apart). */
+int hfb_conv_carry(const float *x, int splits, int x_stride, int x_col0, int taps, float *carried, int64_t slot_stride,
+                   const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, int S, int T, int C, hfb_stream s);
+
+/* Recurrences whose decay is one number per head and token: S <- exp(la) S + c k u^T, o = S^T q + skip u per head; state
+ * [H][dvp][dp] float32 per slot, q, k [T][heads][dp], u [T][H][dvp] in the run's type, zeros in the padding (dp, dvp: d,
+ * dv rounded up to a multiple of 16), o [T][H][dv] float32; la [T][H] (la_stride H) or [H] (la_stride 0), step c [T][H] or
+ * NULL (1), skip [H] or NULL (0); head h reads query/key head h / (H / Hq).
+ * rotate_heads: q, k, u from rows [H q heads | H k heads | H v heads | ..]: rotation (pairs i, i + n_rot / 2), keys times k_scale.
+ * state_space_operands: q, k, u, step, la from rows [z: H dv | x: H dv | B: G d | C: G d | dt: H | ..]: x, B, C through a
+ *   causal convolution with bias and silu (carried inputs as in conv_carry), step = softplus(dt + dt_bias), la = -rate step.
+ * decay_walk: token by token.  decay_chunks: chunks of hfb_decay_chunk_tokens() tokens, bfloat16 operands.
+ * part_norm_gate: rows of o in `parts` equal parts, each divided by its root mean square; silu(g) multiplies before
+ *   (gate_first) or after; times w [C] where given; rows of out out_stride elements apart. */
+int hfb_rotate_heads(const float *src, int splits, int row_stride, const float *cos_sin, int n_rot, int n_positions,
+                     const int32_t *positions, float k_scale, void *q, void *k, void *u, int out_dt, int T, int H, int d, int dv,
+                     int dp, int dvp, hfb_stream s);
+int hfb_state_space_operands(const float *src, int splits, int row_stride, const void *w, int w_dt, const void *bias, int bias_dt,
+                             int taps, const void *dt_bias, int dtb_dt, const float *rate, float *carried, int64_t slot_stride,
+                             const int32_t *token_seq, const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, int S,
+                             void *q, void *k, void *u, int out_dt, float *step, float *la, int T, int H, int G, int d, int dv,
+                             int dp, int dvp, hfb_stream s);
+int hfb_decay_walk(const void *q, const void *k, const void *u, int dt, const float *la, int la_stride, const float *step,
+                   const float *skip, float *state, int64_t slot_stride, const int32_t *cu_tokens, const int32_t *seq_slots,
+                   int n_slots, int S, float *o, int H, int Hq, int d, int dv, int dp, int dvp, hfb_stream s);
+int hfb_decay_chunk_tokens(void);
+size_t hfb_decay_chunks_scratch(int chunks, int H, int dp, int dvp);
+int hfb_decay_chunks(const void *q, const void *k, const void *u, const float *la, int la_stride, const float *step,
+                     const float *skip, float *state, int64_t slot_stride, const int32_t *chunk_t0, const int32_t *chunk_n,
+                     const int32_t *chunk_first, int chunks, const int32_t *seq_slots, int n_slots, int S, void *scratch,
+                     size_t scratch_bytes, float *o, int H, int Hq, int d, int dv, int dp, int dvp, hfb_stream s);
+int hfb_part_norm_gate(const float *o, const float *g, int splits, int g_stride, int g_col0, const float *w, float eps,
+                       int gate_first, void *out, int out_dt, int64_t out_stride, int T, int C, int parts, hfb_stream s);
+
+/* Attention whose queries and keys are normed over the whole projection: the q|k|v|head gates tail (no rotation), and the
+ * gate of one number per head: out[t, h, :] = a[t, h, :] * gate[t, h]. */
+int hfb_row_norm_kv_write(const float *src, int splits, int row_stride, const float *q_w, const float *k_w, float eps,
+                          const int32_t *slots, void *q_out, void *k_cache, void *v_cache, int out_dt, int64_t cache_slots,
+                          float *gate_out, int n_gate, int T, int QD, int KD, int VD, hfb_stream s);
+int hfb_head_gate(const void *a, const float *gate, void *out, int dt, int64_t out_stride, int T, int H, int dv, hfb_stream s);
 
 /* minGRU over a step's tokens: row = `splits` float32 planes [T, 3 W] of [update gate | candidate | output gate] sums;
  * z = sigmoid(a + bz), u = b + bx, cand = u >= 0 ? u + 1/2 : sigmoid(u), S <- (1 - z) S + z cand, out = S silu(g); S [W]

@@ -100,14 +100,14 @@ short_conv_kernel(const float *x, int splits, const void *w, int w_dt, int taps,
 
 // The convolution's carried inputs after a step: the last taps - 1 inputs of each request, from this step's rows and,
 // where the step brought fewer, from what was carried before.  One thread per (request, channel) reads all it needs
-// before it writes.
-__global__ void conv_carry_kernel(const float *x, int splits, int taps, float *carried, size_t slot_stride,
+// before it writes.  Channel c of a row of x is column x_col0 + c of rows x_stride floats apart.
+__global__ void conv_carry_kernel(const float *x, int splits, int x_stride, int x_col0, int taps, float *carried, size_t slot_stride,
                                   const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, int S, int T, int C)
 {
     pdl_entry();
     pdl_sync_small();
     const int K = taps - 1;
-    const size_t plane = (size_t)T * C;
+    const size_t plane = (size_t)T * x_stride;
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < (size_t)S * C; i += (size_t)gridDim.x * blockDim.x) {
         const int seq = (int)(i / C), ch = (int)(i % C);
         const int slot = seq_slots[seq];
@@ -120,7 +120,7 @@ __global__ void conv_carry_kernel(const float *x, int splits, int taps, float *c
             if (j < K) {
                 const int rel = n - K + j;                   // relative to the step's first token of the request
                 float v = 0.f;
-                if (rel >= 0) { for (int s = 0; s < splits; s++) v += x[(size_t)s * plane + (size_t)(t0 + rel) * C + ch]; }
+                if (rel >= 0) { for (int s = 0; s < splits; s++) v += x[(size_t)s * plane + (size_t)(t0 + rel) * x_stride + x_col0 + ch]; }
                 else v = st[(size_t)(rel + K) * C + ch];
                 keep[j] = v;
             }
@@ -449,6 +449,17 @@ extern "C" int hfb_decay(const float *z, int splits, int z_stride, int z_col0, c
     return check_pdl_launch(g_launch_err, "decay");
 }
 
+extern "C" int hfb_conv_carry(const float *x, int splits, int x_stride, int x_col0, int taps, float *carried, int64_t slot_stride,
+                              const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, int S, int T, int C, hfb_stream s)
+{
+    if (T <= 0 || S <= 0 || taps <= 1) return HFB_OK;
+    if (!x || !carried || !cu_tokens || !seq_slots || splits < 1 || x_col0 < 0 || x_col0 + C > x_stride || taps > CONV_MAX_TAPS)
+        return fail(HFB_EINVAL, "conv_carry: bad arguments (taps=%d C=%d)", taps, C);
+    g_launch_err = launch_pdl(conv_carry_kernel, dim3(rec_blocks((size_t)S * C)), dim3(256), 0, (cudaStream_t)s, x, splits, x_stride, x_col0,
+                              taps, carried, (size_t)slot_stride, cu_tokens, seq_slots, n_slots, S, T, C);
+    return check_pdl_launch(g_launch_err, "conv_carry");
+}
+
 extern "C" int hfb_short_conv(const float *x, int splits, const void *w, int w_dt, int taps, float *carried, int64_t slot_stride,
                               const int32_t *token_seq, const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, int S,
                               float *out, int T, int n_a, int d_a, int n_b, int d_b, int n_unit, int n_scaled, float scale,
@@ -467,9 +478,7 @@ extern "C" int hfb_short_conv(const float *x, int splits, const void *w, int w_d
     int rc = check_pdl_launch(g_launch_err, "short_conv");
     if (rc != HFB_OK || taps == 1) return rc;
     const int C = n_a * d_a + n_b * d_b;
-    g_launch_err = launch_pdl(conv_carry_kernel, dim3(rec_blocks((size_t)S * C)), dim3(256), 0, (cudaStream_t)s, x, splits, taps, carried,
-                              (size_t)slot_stride, cu_tokens, seq_slots, n_slots, S, T, C);
-    return check_pdl_launch(g_launch_err, "conv_carry");
+    return hfb_conv_carry(x, splits, C, 0, taps, carried, slot_stride, cu_tokens, seq_slots, n_slots, S, T, C, s);
 }
 
 extern "C" int hfb_linear_scan(const float *q, int q_stride, const float *k, int k_stride, const float *v, int v_stride,

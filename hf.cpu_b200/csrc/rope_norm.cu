@@ -130,9 +130,166 @@ rope_norm_kv_kernel(const float *src, int splits, const void *bias, int bias_dt,
     else { for (int c = lane; c < n; c += 32) dst[c] = from_f32<TO>(x[c] * r); }
 }
 
+// The tail for attention whose queries and keys are normed over the whole projection (all heads at once) before the heads
+// are told apart, without rotation: row = [QD queries | KD keys | VD values | n_gate head gates | ...], row_stride floats,
+// `splits` planes.  q = row / sqrt(mean(row^2) + eps) * q_w over the QD queries, keys likewise with k_w; queries to q_out
+// [T, QD], keys and values to the token's cache slot (KD = VD = 0: the layer reads another layer's cache), gates as
+// sigmoid(row) to gate_out [T, n_gate] float32.  One block per token.
+__device__ __forceinline__ float4 sum_planes4(const float *p, int splits, size_t plane)
+{
+    float4 a = *(const float4 *)p;
+    for (int s = 1; s < splits; s++) {
+        const float4 b = *(const float4 *)(p + (size_t)s * plane);
+        a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
+    }
+    return a;
+}
+
+__device__ __forceinline__ float sum_planes(const float *p, int splits, size_t plane)
+{
+    float a = *p;
+    for (int s = 1; s < splits; s++) a += p[(size_t)s * plane];
+    return a;
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(256)
+row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_w, const float *k_w, float eps, const int32_t *slots,
+                   TO *q_out, TO *k_cache, TO *v_cache, long long cache_slots, float *gate_out, int n_gate, int T, int QD, int KD, int VD,
+                   int vec, int *err)
+{
+    pdl_entry();
+    pdl_sync_small();
+    extern __shared__ __align__(16) float rn_row[];                      // [QD + KD]
+    __shared__ float red[16];
+    const int t = blockIdx.x, n = QD + KD;
+    const size_t plane = (size_t)T * row_stride;
+    const float *row = src + (size_t)t * row_stride;
+    long long slot = (KD + VD > 0 && slots) ? slots[t] : -1;
+    if (slot >= cache_slots) { if (threadIdx.x == 0) atomicOr(err, HFB_ERR_SLOT); slot = -1; }
+    float sq = 0.f, sk = 0.f;
+    if (vec) {
+        for (int c = threadIdx.x * 4; c < n; c += 1024) {
+            const float4 v = sum_planes4(row + c, splits, plane);
+            *(float4 *)(rn_row + c) = v;
+            const float ss = (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+            if (c < QD) sq += ss; else sk += ss;
+        }
+        if (slot >= 0)
+            for (int c = threadIdx.x * 4; c < VD; c += 1024) store4(v_cache + (size_t)slot * VD + c, sum_planes4(row + n + c, splits, plane));
+    } else {
+        for (int c = threadIdx.x; c < n; c += 256) {
+            const float v = sum_planes(row + c, splits, plane);
+            rn_row[c] = v;
+            if (c < QD) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
+        }
+        if (slot >= 0)
+            for (int c = threadIdx.x; c < VD; c += 256) v_cache[(size_t)slot * VD + c] = from_f32<TO>(sum_planes(row + n + c, splits, plane));
+    }
+    for (int c = threadIdx.x; c < n_gate; c += 256)
+        gate_out[(size_t)t * n_gate + c] = 1.0f / (1.0f + expf(-sum_planes(row + n + VD + c, splits, plane)));
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (lane == 0) { red[warp] = sq; red[8 + warp] = sk; }
+    __syncthreads();
+    sq = warp_sum(lane < 8 ? red[lane] : 0.f);
+    sk = warp_sum(lane < 8 ? red[8 + lane] : 0.f);
+    const float rq = 1.0f / sqrtf(sq / (float)QD + eps), rk = 1.0f / sqrtf(sk / (float)max(KD, 1) + eps);
+    TO *qo = q_out + (size_t)t * QD, *ko = k_cache + (size_t)(slot < 0 ? 0 : slot) * KD;
+    if (vec) {
+        for (int c = threadIdx.x * 4; c < n; c += 1024) {
+            const bool is_q = c < QD;
+            if (!is_q && slot < 0) continue;
+            const float4 w = *(const float4 *)(is_q ? q_w + c : k_w + (c - QD));
+            const float r = is_q ? rq : rk;
+            float4 v = *(const float4 *)(rn_row + c);
+            v.x *= r * w.x; v.y *= r * w.y; v.z *= r * w.z; v.w *= r * w.w;
+            store4(is_q ? qo + c : ko + (c - QD), v);
+        }
+    } else {
+        for (int c = threadIdx.x; c < n; c += 256) {
+            if (c < QD) qo[c] = from_f32<TO>(rn_row[c] * rq * q_w[c]);
+            else if (slot >= 0) ko[c - QD] = from_f32<TO>(rn_row[c] * rk * k_w[c - QD]);
+        }
+    }
+}
+
+// out[t, h, :] = a[t, h, :] * gate[t, h], rows of out `out_stride` elements apart.
+template <typename T_>
+__global__ void head_gate_kernel(const T_ *a, const float *gate, T_ *out, size_t out_stride, int T, int H, int dv, int vec)
+{
+    pdl_entry();
+    pdl_sync_small();
+    const int C = H * dv;
+    if (vec) {
+        const size_t total = (size_t)T * C / 4;
+        const int per = C / 4;
+        for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+            const size_t t = i / per;
+            const int c = (int)(i - t * per) * 4;
+            const float g = gate[t * H + c / dv];
+            const T_ *p = a + t * C + c;
+            store4(out + t * out_stride + c, make_float4(to_f32(p[0]) * g, to_f32(p[1]) * g, to_f32(p[2]) * g, to_f32(p[3]) * g));
+        }
+    } else {
+        const size_t total = (size_t)T * C;
+        for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+            const size_t t = i / C;
+            const int c = (int)(i - t * C);
+            out[t * out_stride + c] = from_f32<T_>(to_f32(a[i]) * gate[t * H + c / dv]);
+        }
+    }
+}
+
 }  // namespace hfb
 
 using namespace hfb;
+
+extern "C" int hfb_row_norm_kv_write(const float *src, int splits, int row_stride, const float *q_w, const float *k_w, float eps,
+                                     const int32_t *slots, void *q_out, void *k_cache, void *v_cache, int out_dt, int64_t cache_slots,
+                                     float *gate_out, int n_gate, int T, int QD, int KD, int VD, hfb_stream s)
+{
+    if (T <= 0) return HFB_OK;
+    if (!src || splits < 1 || QD <= 0 || KD < 0 || VD < 0 || n_gate < 0 || row_stride < QD + KD + VD + n_gate || !q_w || (KD && !k_w) || !q_out ||
+        !valid_dt(out_dt) || (n_gate && !gate_out) || (slots && KD && (!k_cache || !v_cache)))
+        return fail(HFB_EINVAL, "row_norm_kv_write: bad arguments (QD=%d KD=%d VD=%d)", QD, KD, VD);
+    const size_t smem = (size_t)(QD + KD) * sizeof(float);
+    if (smem > 200 * 1024) return fail(HFB_ENOTSUP, "row_norm_kv_write: %d query and key channels exceed %d", QD + KD, 50 * 1024);
+    const int esz = out_dt == HFB_F32 ? 4 : 2;
+    auto al = [](const void *p, int b) { return ((uintptr_t)p & (b - 1)) == 0; };
+    const int vec = ((QD | KD | VD | row_stride) & 3) == 0 && al(src, 16) && al(q_w, 16) && al(k_w, 16) && al(q_out, 4 * esz) &&
+                    al(k_cache, 4 * esz) && al(v_cache, 4 * esz);
+#define HFB_RNK(TY) do { \
+        if (smem > 48 * 1024) { \
+            cudaError_t e = cudaFuncSetAttribute(row_norm_kv_kernel<TY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return fail(HFB_ECUDA, "row_norm_kv_write: %s", cudaGetErrorString(e)); \
+        } \
+        g_launch_err = launch_pdl(row_norm_kv_kernel<TY>, dim3(T), dim3(256), smem, (cudaStream_t)s, src, splits, row_stride, q_w, k_w, eps, slots, \
+            (TY *)q_out, (TY *)k_cache, (TY *)v_cache, (long long)cache_slots, gate_out, n_gate, T, QD, KD, VD, vec, error_word()); \
+    } while (0)
+    if (out_dt == HFB_F32) HFB_RNK(float);
+    else HFB_RNK(__nv_bfloat16);
+#undef HFB_RNK
+    return check_pdl_launch(g_launch_err, "row_norm_kv_write");
+}
+
+extern "C" int hfb_head_gate(const void *a, const float *gate, void *out, int dt, int64_t out_stride, int T, int H, int dv, hfb_stream s)
+{
+    if (T <= 0) return HFB_OK;
+    if (!a || !gate || !out || !valid_dt(dt) || H <= 0 || dv <= 0 || out_stride < (int64_t)H * dv) return fail(HFB_EINVAL, "head_gate: bad arguments");
+    const int esz = dt == HFB_F32 ? 4 : 2;
+    const int vec = (dv & 3) == 0 && (out_stride & 3) == 0 && ((uintptr_t)a & (4 * esz - 1)) == 0 && ((uintptr_t)out & (4 * esz - 1)) == 0;
+    const size_t work = (size_t)T * H * dv / (vec ? 4 : 1);
+    const unsigned blocks = (unsigned)((work + 255) / 256 < 148 * 16 ? (work + 255) / 256 : 148 * 16);
+    if (dt == HFB_F32)
+        g_launch_err = launch_pdl(head_gate_kernel<float>, dim3(blocks), dim3(256), 0, (cudaStream_t)s, (const float *)a, gate, (float *)out,
+                                  (size_t)out_stride, T, H, dv, vec);
+    else
+        g_launch_err = launch_pdl(head_gate_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, (cudaStream_t)s, (const __nv_bfloat16 *)a, gate,
+                                  (__nv_bfloat16 *)out, (size_t)out_stride, T, H, dv, vec);
+    return check_pdl_launch(g_launch_err, "head_gate");
+}
 
 extern "C" int hfb_rope_norm_kv_write(const float *src, int splits, const void *bias, int bias_dt, const float *cos_sin,
                                       int n_rot, int n_positions, const int32_t *positions, const int32_t *slots,

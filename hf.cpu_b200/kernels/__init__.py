@@ -283,6 +283,7 @@ def linear_rope_kv(a, w, bias, qkv_buf, cos_sin, n_rot, positions, slots, q_out,
     backend().linear_rope_kv(a, w, bias, qkv_buf, cos_sin, int(n_rot), positions, slots, q_out, k_cache, v_cache, H, G, d)
 
 
+ACT_CLAMPED_GLU = 5          # a gated pair only: see linear_glu
 ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2, "relu2": 3, "none": 4}       # relu2: the square of relu
 ACT_GLU = 256               # added to an activation code: gated form of the grouped product
 MOE_TILE = 128              # places of one expert per tile of the grouped product ...
@@ -460,14 +461,23 @@ def headwise_linear(x, w, out, H: int, in_row: int, out_row: int) -> None:
     backend().headwise_linear(x, w, out, int(H), int(in_row), int(out_row))
 
 
-def linear_glu(a: torch.Tensor, w: torch.Tensor, gu_buf: torch.Tensor, out: torch.Tensor, act: str) -> None:
-    """out = act(g) * u where [g0, u0, g1, u1, ...] = a @ w.T (rows of ``w`` alternate gate, up)."""
+def linear_glu(a: torch.Tensor, w: torch.Tensor, gu_buf: torch.Tensor, out: torch.Tensor, act: str, bias=None, clamp=None) -> None:
+    """out = act(g) * u where [g0, u0, g1, u1, ...] = a @ w.T + bias (rows of ``w`` and entries of ``bias`` alternate gate,
+    up).  act "clamped" with ``clamp`` = (limit, alpha, offset): g = min(g, limit), u = clamp(u, -limit, limit), out = g *
+    sigmoid(alpha g) * (u + offset).  ``out`` may be a column slice of a wider array."""
     _need(a.shape[1] == w.shape[1] and w.shape[0] == 2 * out.shape[1] and out.shape[0] == a.shape[0], "linear_glu: shape mismatch")
     _need(gu_buf.shape == (a.shape[0], w.shape[0]), "linear_glu: scratch must be [M, 2F]")
-    if act == "silu":
+    _need(out.stride(1) == 1 and (bias is None or bias.shape == (w.shape[0],)), "linear_glu: out has unit column stride, bias is [2F]")
+    _need((act == "clamped") == (clamp is not None), "linear_glu: the clamped form and its constants come together")
+    if act == "silu" and bias is None and out.is_contiguous():
         backend().linear_swiglu(a, w, gu_buf, out)
-    else:
-        backend().linear_glu(a, w, gu_buf, out, _act(act))
+        return
+    extra = {}
+    if bias is not None:
+        extra["bias"] = bias
+    if clamp is not None:
+        extra["clamp"] = tuple(float(x) for x in clamp)
+    backend().linear_glu(a, w, gu_buf, out, ACT_CLAMPED_GLU if act == "clamped" else _act(act), **extra)
 
 
 def linear_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str) -> None:
@@ -479,6 +489,12 @@ def linear_act(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str) ->
 def scale_(x: torch.Tensor, s: float) -> None:
     _need(x.dtype == torch.float32 and x.is_contiguous(), "scale_: float32, contiguous")
     backend().scale_(x, float(s))
+
+
+def softcap_(x: torch.Tensor, cap: float) -> None:
+    """x = cap * tanh(x / cap)."""
+    _need(x.dtype == torch.float32 and x.is_contiguous() and cap > 0, "softcap_: float32, contiguous; a positive cap")
+    backend().softcap_(x, float(cap))
 
 
 def moe_route(h, w, b, top: int, ids, weights, logits) -> None:
@@ -669,6 +685,123 @@ def gate_norm(o, w, eps: float, g, g_splits: int, g_stride: int, g_col0: int, ga
     _need(g.dtype == torch.float32 and g.numel() >= g_splits * T * g_stride and g_col0 + H * dv <= g_stride and gate in ("silu", "sigmoid"),
           "gate_norm: g float32 [splits, T, stride]; gate silu or sigmoid")
     backend().gate_norm(o, w, float(eps), g, int(g_splits), int(g_stride), int(g_col0), 0 if gate == "silu" else 1, out, int(H), int(dv))
+
+
+# ---- recurrences with one decay per head and token ---------------------------------------------------------------
+DECAY_CHUNK = 64            # tokens of a chunk of the chunked form
+DECAY_CHUNK_MIN = 16        # steps whose longest portion is shorter walk token by token
+
+
+def padded_head(d: int) -> int:
+    """A head's size in the operands and the state of :func:`decay_scan`: rounded up to a multiple of 16."""
+    return (int(d) + 15) // 16 * 16
+
+
+def decay_chunk_arrays(q_lens):
+    """The chunks of a step's tokens for :func:`decay_scan` as named int32 arrays: first token (``t0``) and count (``n``) of
+    every chunk, and every request's first chunk (``first``, one more at the end); none for a step of short portions."""
+    import numpy as np
+    if max(q_lens) < DECAY_CHUNK_MIN:
+        return {}
+    t0, n, first, at = [], [], [0], 0
+    for m in q_lens:
+        for a in range(0, m, DECAY_CHUNK):
+            t0.append(at + a)
+            n.append(min(DECAY_CHUNK, m - a))
+        at += m
+        first.append(len(t0))
+    return {"t0": np.asarray(t0, dtype=np.int32), "n": np.asarray(n, dtype=np.int32), "first": np.asarray(first, dtype=np.int32)}
+
+
+def _decay_ok(q, k, u, H, Hq, d, dv, what):
+    T, dp, dvp = q.shape[0], padded_head(d), padded_head(dv)
+    _need(H % Hq == 0 and q.shape == k.shape == (T, Hq * dp) and u.shape == (T, H * dvp) and q.dtype == k.dtype == u.dtype,
+          f"{what}: q, k are [T, Hq * padded d], u [T, H * padded dv], of one type")
+    _need(dp <= SCAN_MAX_HEAD, f"{what}: key heads above {SCAN_MAX_HEAD} are not supported")
+
+
+def rotate_heads(src, splits: int, row: int, cos_sin, n_rot: int, positions, k_scale: float, q, k, u, H: int, d: int, dv: int) -> None:
+    """Operands of retention from the sums of its product (``splits`` float32 planes [T, row]: H query heads of d, H key
+    heads of d, H value heads of dv, ...): rotation of the first ``n_rot`` dimensions (i with i + n_rot/2) of queries and
+    keys, keys times ``k_scale``; q, k, u as :func:`decay_scan` takes them."""
+    _decay_ok(q, k, u, H, H, d, dv, "rotate_heads")
+    _need(src.dtype == torch.float32 and src.numel() >= splits * q.shape[0] * row and row >= H * (2 * d + dv), "rotate_heads: rows are float32 [splits, T, row]")
+    _need(n_rot % 2 == 0 and 0 <= n_rot <= d and (n_rot == 0 or (cos_sin is not None and cos_sin.shape[1:] == (n_rot // 2, 2)
+          and cos_sin.dtype == torch.float32)), "rotate_heads: cos/sin table must be float32 [positions, n_rot/2, 2]")
+    backend().rotate_heads(src, int(splits), int(row), cos_sin, int(n_rot), positions, float(k_scale), q, k, u, int(H), int(d), int(dv))
+
+
+def state_space_operands(src, splits: int, row: int, conv_w, conv_b, dt_bias, rate, carried, ctx, q, k, u, step, la, H: int, G: int,
+                         d: int, dv: int) -> None:
+    """Operands of the state-space recurrence from the sums of its product (``splits`` float32 planes [T, row]: z of H * dv,
+    x of H * dv, B of G * d, C of G * d, dt of H, ...).  x, B and C pass a causal convolution per channel (``conv_w`` [C,
+    taps], last column the current token's, bias ``conv_b``) and silu and become u, k and q; ``carried`` [slots, taps - 1, C]
+    float32 holds each request's last inputs and is brought up to date.  step = softplus(dt + dt_bias), la = -rate * step
+    (float32 [T, H])."""
+    _decay_ok(q, k, u, H, G, d, dv, "state_space_operands")
+    T, C, taps = q.shape[0], H * dv + 2 * G * d, conv_w.shape[1]
+    _need(src.dtype == torch.float32 and src.numel() >= splits * T * row and row >= H * dv + C + H, "state_space_operands: rows are float32 [splits, T, row]")
+    _need(conv_w.shape == (C, taps) and 1 <= taps <= CONV_MAX_TAPS and conv_b.shape == (C,), "state_space_operands: channel count or taps mismatch")
+    _need(dt_bias.shape == (H,) and rate.shape == (H,) and rate.dtype == torch.float32, "state_space_operands: dt_bias [H], rate float32 [H]")
+    _need(carried.dtype == torch.float32 and carried.dim() == 3 and carried.shape[1:] == (max(taps - 1, 1), C)
+          and carried.stride()[1:] == (C, 1), "state_space_operands: carried is float32 [slots, taps - 1, C]")
+    _need(step.shape == la.shape == (T, H) and step.dtype == la.dtype == torch.float32, "state_space_operands: step and la are float32 [T, H]")
+    backend().state_space_operands(src, int(splits), int(row), conv_w, conv_b, dt_bias, rate, carried, ctx, q, k, u, step, la, int(H), int(G),
+                                   int(d), int(dv))
+
+
+def decay_scan(q, k, u, la, step, skip, state, ctx, o, H: int, Hq: int, d: int, dv: int, chunks=None) -> None:
+    """Per head, along each request's tokens from its slot's state: S <- exp(la) S + step k u^T, o = S^T q + skip u.  q, k [T,
+    Hq heads], u [T, H heads] with heads padded with zeros to :func:`padded_head`; ``la`` float32 [T, H], or [H] for a decay
+    that is the same for every token; ``step`` float32 [T, H] or None (1); ``skip`` float32 [H] or None; ``state`` float32
+    [slots, H, padded dv, padded d]; ``o`` float32 [T, H * dv].  ``chunks``: the device arrays of :func:`decay_chunk_arrays`
+    for this step (empty or None: the walk)."""
+    _decay_ok(q, k, u, H, Hq, d, dv, "decay_scan")
+    T, dp, dvp = q.shape[0], padded_head(d), padded_head(dv)
+    _need(la.dtype == torch.float32 and la.shape in ((T, H), (H,)), "decay_scan: la is float32 [T, H] or [H]")
+    _need(step is None or (step.dtype == torch.float32 and step.shape == (T, H)), "decay_scan: step is float32 [T, H]")
+    _need(skip is None or (skip.dtype == torch.float32 and skip.shape == (H,)), "decay_scan: skip is float32 [H]")
+    _need(state.dtype == torch.float32 and state.shape[1:] == (H, dvp, dp) and state.stride()[1:] == (dvp * dp, dp, 1)
+          and state.stride(0) % 4 == 0, "decay_scan: state is float32 [slots, H, padded dv, padded d], slots a multiple of four apart")
+    _need(o.shape == (T, H * dv) and o.dtype == torch.float32, "decay_scan: o is float32 [T, H * dv]")
+    backend().decay_scan(q, k, u, la, step, skip, state, ctx, o, int(H), int(Hq), int(d), int(dv), chunks or {})
+
+
+def part_norm_gate(o, parts: int, eps: float, g, g_splits: int, g_stride: int, g_col0: int, w, gate_first: bool, out) -> None:
+    """out = the rows of o (float32 [T, C]) in ``parts`` equal parts, each divided by its own root mean square, times ``w``
+    (float32 [C]) where given; silu(g) multiplies before the norm (``gate_first``) or after it, g the sum of ``g_splits``
+    float32 planes [T, g_stride] read from column ``g_col0`` on.  ``out`` may be a column slice of a wider array."""
+    T, C = o.shape
+    _need(o.dtype == torch.float32 and out.shape == (T, C) and out.stride(1) == 1 and C % parts == 0, "part_norm_gate: shape mismatch")
+    _need(g.dtype == torch.float32 and g.numel() >= g_splits * T * g_stride and g_col0 + C <= g_stride, "part_norm_gate: g is float32 [splits, T, stride]")
+    _need(w is None or (w.shape == (C,) and w.dtype == torch.float32), "part_norm_gate: the weight is float32 [C]")
+    backend().part_norm_gate(o, int(parts), float(eps), g, int(g_splits), int(g_stride), int(g_col0), w, bool(gate_first), out)
+
+
+# ---- attention normed over the whole projection, head gates -------------------------------------------------------
+def linear_row_norm_kv(a, w, buf, q_w, k_w, eps: float, slots, q_out, k_cache, v_cache, gate_out, H: int, G: int, d: int, dv: int) -> None:
+    """The q|k|v|head gates product and its tail for attention whose queries and keys are rms-normed over the whole
+    projection, without rotation: row = a @ w.T = [H * d | G * d | G * dv | gates of gate_out | ...] (G = 0: no keys and values of
+    its own); queries x / sqrt(mean(x^2) + eps) * q_w to ``q_out``, keys likewise (k_w) and values to the cache at ``slots``,
+    sigmoid of the gates to ``gate_out`` (float32 [T, H]).  ``buf`` [T, row] float32 is scratch."""
+    T, C = a.shape[0], w.shape[0]
+    _need(a.shape[1] == w.shape[1] and buf.shape == (T, C) and buf.dtype == torch.float32, "linear_row_norm_kv: scratch must be float32 [T, row]")
+    _need(gate_out is None or (gate_out.shape[0] == T and gate_out.dtype == torch.float32), "linear_row_norm_kv: gates are float32 [T, heads]")
+    n_gate = 0 if gate_out is None else gate_out.shape[1]
+    _need(C >= H * d + G * (d + dv) + n_gate and q_out.shape == (T, H * d), "linear_row_norm_kv: shape mismatch")
+    _need(q_w.shape == (H * d,) and q_w.dtype == torch.float32 and (G == 0 or (k_w.shape == (G * d,) and k_w.dtype == torch.float32)),
+          "linear_row_norm_kv: norm weights are float32 over the whole projection")
+    if G:
+        _need(k_cache.shape[2:] == (G, d) and v_cache.shape[2:] == (G, dv) and k_cache.dtype == v_cache.dtype == q_out.dtype,
+              "linear_row_norm_kv: cache geometry mismatch")
+    backend().linear_row_norm_kv(a, w, buf, q_w, k_w, float(eps), slots, q_out, k_cache, v_cache, gate_out, int(H), int(G), int(d), int(dv))
+
+
+def head_gate(a, gate, out, H: int, dv: int) -> None:
+    """out[t, h] = a[t, h] * gate[t, h]; a [T, H * dv], gate float32 [T, H]; ``out`` may be a column slice of a wider array."""
+    _need(a.shape == out.shape and a.shape[1] == H * dv and a.dtype == out.dtype and out.stride(1) == 1, "head_gate: a and out must agree")
+    _need(gate.dtype == torch.float32 and gate.shape == (a.shape[0], H), "head_gate: gates are float32 [T, H]")
+    backend().head_gate(a, gate, out, int(H), int(dv))
 
 
 # ---- layer norm, token shift, gates, minGRU ----------------------------------------------------------------------

@@ -74,6 +74,11 @@ class NativeBackend:
         self._counters = None
         self.lib.hfb_linear_tc_partials_workspace.restype = ctypes.c_size_t
         self.lib.hfb_argmax2_scratch.restype = ctypes.c_size_t
+        self.lib.hfb_decay_chunks_scratch.restype = ctypes.c_size_t
+        from . import DECAY_CHUNK
+        if self.lib.hfb_decay_chunk_tokens() != DECAY_CHUNK:
+            raise KernelError("the library's chunks and the binding's are not of one length")
+        self.decay_chunks = os.environ.get("HFB_DECAY_CHUNKS", "1") != "0"     # portions of a recurrence with scalar decays in chunks
         self.path = path
         self.launches = 0          # kernels launched through this binding (one per successful call)
 
@@ -93,6 +98,13 @@ class NativeBackend:
         for t in ts:
             if t is not None and (not t.is_cuda or not t.is_contiguous()):
                 raise KernelError("kernel arguments must be contiguous CUDA tensors")
+
+    @staticmethod
+    def _rows_on_gpu(*ts):
+        """Arrays whose rows are contiguous; they may be column slices of wider ones."""
+        for t in ts:
+            if not t.is_cuda or t.dim() != 2 or t.stride(1) != 1 or t.stride(0) < t.shape[1]:
+                raise KernelError("kernel outputs must be CUDA tensors with contiguous rows")
 
     # ---- entry points -------------------------------------------------------------------------
     def embed(self, ids, table, out):
@@ -465,17 +477,21 @@ class NativeBackend:
                                                  c_int(H), c_int(w.shape[1]), c_int(w.shape[2]), c_int(in_row), c_int(out_row),
                                                  self._stream()), "headwise_linear")
 
-    def linear_glu(self, a, w, gu_buf, out, act):
-        self._on_gpu(a, w, gu_buf, out)
+    def linear_glu(self, a, w, gu_buf, out, act, bias=None, clamp=None):
+        self._on_gpu(a, w, bias)
+        self._rows_on_gpu(out)
+        b_dt = c_int(_dt(bias) if bias is not None else 0)
+        consts = tuple(c_float(x) for x in (clamp or (0.0, 0.0, 0.0)))
+        ldo = c_int64(out.stride(0))
         if self._tc_ok(a, w, out):
             M, K = a.shape
-            self._check(self.lib.hfb_linear_tc_glu(_p(a), _p(w), _p(out), c_int(_dt(out)), c_int(M), c_int(w.shape[0]), c_int(K),
-                                                   c_int(act), self._stream()), "linear_tc_glu")
+            self._check(self.lib.hfb_linear_tc_glu(_p(a), _p(w), _p(bias), b_dt, _p(out), c_int(_dt(out)), ldo, c_int(M), c_int(w.shape[0]),
+                                                   c_int(K), c_int(act), *consts, self._stream()), "linear_tc_glu")
             return
         self.linear(a, w, None, gu_buf, False)
         T, F = out.shape
-        self._check(self.lib.hfb_glu(_p(gu_buf), _p(out), c_int(_dt(out)), c_int(T), c_int(F), c_int(1), c_int(act),
-                                     self._stream()), "glu")
+        self._check(self.lib.hfb_glu(_p(gu_buf), _p(bias), b_dt, _p(out), c_int(_dt(out)), ldo, c_int(T), c_int(F), c_int(1), c_int(act),
+                                     *consts, self._stream()), "glu")
 
     def linear_act(self, a, w, out, act):
         self._on_gpu(a, w, out)
@@ -490,6 +506,10 @@ class NativeBackend:
     def scale_(self, x, s):
         self._on_gpu(x)
         self._check(self.lib.hfb_scale(_p(x), c_int64(x.numel()), c_float(s), self._stream()), "scale")
+
+    def softcap_(self, x, cap):
+        self._on_gpu(x)
+        self._check(self.lib.hfb_softcap(_p(x), c_int64(x.numel()), c_float(cap), self._stream()), "softcap")
 
     def moe_route(self, h, w, b, top, ids, weights, logits):
         self._on_gpu(h, w, b, ids, weights, logits)
@@ -572,6 +592,66 @@ class NativeBackend:
         self._check(self.lib.hfb_gate_norm(_p(o), _p(w), c_int(_dt(w)), c_float(eps), _p(g), c_int(g_splits), c_int(g_stride),
                                            c_int(g_col0), c_int(gate), _p(out), c_int(_dt(out)), c_int(o.shape[0]), c_int(H), c_int(dv),
                                            self._stream()), "gate_norm")
+
+    def rotate_heads(self, src, splits, row, cos_sin, n_rot, positions, k_scale, q, k, u, H, d, dv):
+        self._on_gpu(src, cos_sin, positions, q, k, u)
+        self._check(self.lib.hfb_rotate_heads(
+            _p(src), c_int(splits), c_int(row), _p(cos_sin), c_int(n_rot), c_int(cos_sin.shape[0] if cos_sin is not None else 0), _p(positions),
+            c_float(k_scale), _p(q), _p(k), _p(u), c_int(_dt(q)), c_int(q.shape[0]), c_int(H), c_int(d), c_int(dv), c_int(q.shape[1] // H),
+            c_int(u.shape[1] // H), self._stream()), "rotate_heads")
+
+    def state_space_operands(self, src, splits, row, conv_w, conv_b, dt_bias, rate, carried, ctx, q, k, u, step, la, H, G, d, dv):
+        self._on_gpu(src, conv_w, conv_b, dt_bias, rate, q, k, u, step, la, ctx.token_seq, ctx.cu_tokens, ctx.seq_slots)
+        taps = conv_w.shape[1]
+        self._check(self.lib.hfb_state_space_operands(
+            _p(src), c_int(splits), c_int(row), _p(conv_w), c_int(_dt(conv_w)), _p(conv_b), c_int(_dt(conv_b)), c_int(taps), _p(dt_bias),
+            c_int(_dt(dt_bias)), _p(rate), _p(carried), c_int64(carried.stride(0)), _p(ctx.token_seq), _p(ctx.cu_tokens), _p(ctx.seq_slots),
+            c_int(carried.shape[0]), c_int(ctx.num_seqs), _p(q), _p(k), _p(u), c_int(_dt(q)), _p(step), _p(la), c_int(q.shape[0]), c_int(H),
+            c_int(G), c_int(d), c_int(dv), c_int(q.shape[1] // G), c_int(u.shape[1] // H), self._stream()), "state_space_operands")
+        if taps > 1 and q.shape[0] != ctx.num_seqs:
+            self.launches += 1
+
+    def decay_scan(self, q, k, u, la, step, skip, state, ctx, o, H, Hq, d, dv, chunks):
+        self._on_gpu(q, k, u, la, step, skip, o, ctx.cu_tokens, ctx.seq_slots)
+        dp, dvp = q.shape[1] // Hq, u.shape[1] // H
+        la_stride = H if la.dim() == 2 else 0
+        if chunks and self.decay_chunks and q.dtype == torch.bfloat16:
+            t0, n, first = chunks["t0"], chunks["n"], chunks["first"]
+            need = self.lib.hfb_decay_chunks_scratch(c_int(t0.shape[0]), c_int(H), c_int(dp), c_int(dvp))
+            if need:
+                scratch = ctx.buf("decay_chunks", (need,), torch.uint8)
+                self._check(self.lib.hfb_decay_chunks(
+                    _p(q), _p(k), _p(u), _p(la), c_int(la_stride), _p(step), _p(skip), _p(state), c_int64(state.stride(0)), _p(t0), _p(n), _p(first),
+                    c_int(t0.shape[0]), _p(ctx.seq_slots), c_int(state.shape[0]), c_int(ctx.num_seqs), _p(scratch), ctypes.c_size_t(need), _p(o),
+                    c_int(H), c_int(Hq), c_int(d), c_int(dv), c_int(dp), c_int(dvp), self._stream()), "decay_chunks")
+                self.launches += 2
+                return
+        self._check(self.lib.hfb_decay_walk(
+            _p(q), _p(k), _p(u), c_int(_dt(q)), _p(la), c_int(la_stride), _p(step), _p(skip), _p(state), c_int64(state.stride(0)), _p(ctx.cu_tokens),
+            _p(ctx.seq_slots), c_int(state.shape[0]), c_int(ctx.num_seqs), _p(o), c_int(H), c_int(Hq), c_int(d), c_int(dv), c_int(dp), c_int(dvp),
+            self._stream()), "decay_walk")
+
+    def part_norm_gate(self, o, parts, eps, g, g_splits, g_stride, g_col0, w, gate_first, out):
+        self._on_gpu(o, g, w)
+        self._rows_on_gpu(out)
+        self._check(self.lib.hfb_part_norm_gate(
+            _p(o), _p(g), c_int(g_splits), c_int(g_stride), c_int(g_col0), _p(w), c_float(eps), c_int(1 if gate_first else 0), _p(out),
+            c_int(_dt(out)), c_int64(out.stride(0)), c_int(o.shape[0]), c_int(o.shape[1]), c_int(parts), self._stream()), "part_norm_gate")
+
+    def linear_row_norm_kv(self, a, w, buf, q_w, k_w, eps, slots, q_out, k_cache, v_cache, gate_out, H, G, d, dv):
+        self._on_gpu(a, w, buf, q_w, k_w, slots, q_out, k_cache, v_cache, gate_out)
+        src, splits = self._product_sums(a, w, buf)
+        self._check(self.lib.hfb_row_norm_kv_write(
+            _p(src), c_int(splits), c_int(w.shape[0]), _p(q_w), _p(k_w if G else None), c_float(eps), _p(slots if G else None), _p(q_out),
+            _p(k_cache if G else None), _p(v_cache if G else None), c_int(_dt(q_out)), c_int64(k_cache.shape[0] * k_cache.shape[1] if G else 0),
+            _p(gate_out), c_int(gate_out.shape[1] if gate_out is not None else 0), c_int(a.shape[0]), c_int(H * d), c_int(G * d), c_int(G * dv),
+            self._stream()), "row_norm_kv_write")
+
+    def head_gate(self, a, gate, out, H, dv):
+        self._on_gpu(a, gate)
+        self._rows_on_gpu(out)
+        self._check(self.lib.hfb_head_gate(_p(a), _p(gate), _p(out), c_int(_dt(a)), c_int64(out.stride(0)), c_int(a.shape[0]), c_int(H), c_int(dv),
+                                           self._stream()), "head_gate")
 
     def layernorm(self, x, w, eps, center, out, rows):
         self._on_gpu(x, w, out, rows)

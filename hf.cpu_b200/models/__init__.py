@@ -102,6 +102,8 @@ class Model:
             tensors.keep(n for n, c in count.items() if c > 1)
         for part in self.all_parts():
             part.bind(tensors, self.run_dtype, self.device)
+        for l in self.layers:
+            l.block.join_outputs(l.mixer, l.ffn)
         for pos in self.positions.values():
             pos.prepare(self.plan.max_positions, self.device)
         self.bound = True

@@ -28,6 +28,12 @@ rows in the cache).  A rotary encoding with the pairing "interleaved" turns the 
 turns a score s into ``c tanh(s / c)`` (after the factors, before the softmax).  ``out_gate`` = {"tensor": name, "kind":
 "sigmoid" | "silu"}: the concatenated heads' outputs are multiplied element by element by ``kind(W_gate h)`` before the
 output product, ``W_gate`` [H * v_head_dim, hidden] reading the same input as the other projections.
+``qk_row_norm`` = {"q": suffix, "k": suffix} norms queries and keys over the whole projection, all heads at once (``x /
+sqrt(mean(x^2) + qk_norm_eps)`` times a weight as long as the projection), before they are told apart into heads; such a
+layer has no rotation and no biases.  ``head_gate`` names a projection [H, hidden]: head h's output is multiplied by
+``sigmoid(W_gate h)_h``, one number per head, before the output product (with ``qk_row_norm`` only: one product makes q, k, v
+and the gates).  ``cache_window``: the window its cache keeps, where a later layer that reads this layer's cache sees further
+back than this layer does (0: everything).
 """
 from __future__ import annotations
 
@@ -37,7 +43,7 @@ import torch
 
 from .. import kernels
 from ..config.base import UnsupportedError
-from ..weights.loader import TensorSpec, fused_rows
+from ..weights.loader import TensorSpec, fused_rows, pad_rows
 from .base import CacheSpec, Mixer, register_part
 
 
@@ -88,7 +94,8 @@ class PagedAttention(OutputProduct, Mixer):
                  positions=None, names=None, scale=None, v_head_dim=None, qk_norm_eps=None, own_kv: bool = True,
                  bias_suffix: str = ".bias", weight_suffix: str = ".weight", qk_norm_weights=None, chunk: int = 0,
                  v_mix=None, v_mix_tensor: str = "vmix", sink=None, sink_tensor: str = "sink", distance_slope_exp=None,
-                 values_are_keys: bool = False, head_scale_tensor=None, softcap=None, out_gate=None, **_):
+                 values_are_keys: bool = False, head_scale_tensor=None, softcap=None, out_gate=None,
+                 qk_row_norm=None, head_gate=None, cache_window=None, **_):
         self.E, self.H, self.G, self.d = int(hidden_size), int(num_heads), int(num_kv_heads), int(head_dim)
         if self.H % self.G:
             raise UnsupportedError(f"unsupported attention geometry: {self.H} heads over {self.G} key/value heads")
@@ -117,6 +124,15 @@ class PagedAttention(OutputProduct, Mixer):
         self.gate_kind = (out_gate or {}).get("kind", "sigmoid") if out_gate else None
         if self.gate_kind not in (None, "sigmoid", "silu"):
             raise UnsupportedError(f"attention: output gate '{self.gate_kind}' is not known (sigmoid, silu)")
+        self.row_norm = bool(qk_row_norm)
+        if self.row_norm:
+            if self.qk_norm_eps is None or set(qk_row_norm) != {"q", "k"}:
+                raise UnsupportedError("a norm over the whole projection names a weight for q and one for k, and an eps")
+            if position or qkv_bias or v_mix or values_are_keys or qk_norm_weights or out_gate:
+                raise UnsupportedError("a norm over the whole projection goes without rotation, biases, value mixing, keys as values, "
+                                       "head norms and an element-wise output gate")
+        elif head_gate:
+            raise UnsupportedError("a gate per head comes with the norm over the whole projection")
         self.general = (self.qk_norm_eps is not None or self.dv != self.d or not self.own_kv or self.v_mix is not None
                         or self.values_are_keys or self.sink is not None or self.slope_exp is not None
                         or head_scale_tensor is not None or self.softcap > 0 or out_gate is not None
@@ -129,6 +145,9 @@ class PagedAttention(OutputProduct, Mixer):
         self.wsuf, self.bsuf = weight_suffix, bias_suffix
         self.qkv_bias, self.out_bias, self.window = bool(qkv_bias), bool(out_bias), int(window)
         self.mask = kernels.mask_code(self.window, self.chunk)
+        self.cache_window = self.window if cache_window is None else int(cache_window)
+        if self.cache_window and not 0 < self.window <= self.cache_window:
+            raise UnsupportedError("a layer's cache keeps at least the keys its own queries see")
         self.rotary = (positions or {}).get(position) if position else None
         if position and self.rotary is None:
             raise UnsupportedError(f"attention names position encoding '{position}', which the plan does not define")
@@ -145,6 +164,8 @@ class PagedAttention(OutputProduct, Mixer):
         self.gate_name = f"{prefix}.{out_gate['tensor']}" if out_gate else None
         self.sinks = self.slopes = self.head_scales = None          # float32 [H]
         self.w_gate = None
+        self.row_norm_names = {k: f"{prefix}.{v}" for k, v in (qk_row_norm or {}).items()}
+        self.head_gate_name = f"{prefix}.{head_gate}" if head_gate else None
         self.scale = 1.0 / math.sqrt(self.d) if scale is None else float(scale)
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = None
         self.norm_w = None              # (q weight, k weight), float32
@@ -167,7 +188,7 @@ class PagedAttention(OutputProduct, Mixer):
         return self.H * self.dv
 
     def cache_spec(self):
-        return CacheSpec(self.G, self.d, self.window, 0 if self.dv == self.d else self.dv, chunk=self.chunk,
+        return CacheSpec(self.G, self.d, self.cache_window, 0 if self.dv == self.d else self.dv, chunk=self.chunk,
                          values_in_keys=self.values_are_keys)
 
     def step_arrays_key(self):
@@ -191,6 +212,12 @@ class PagedAttention(OutputProduct, Mixer):
         if self.out_bias:
             s.append(TensorSpec(self.names["o"] + self.bsuf, (self.E,)))
         s += [TensorSpec(self.norm_names[x], (self.d,), init="norm") for x in sorted(self.norm_names)]
+        if self.row_norm:
+            s.append(TensorSpec(self.row_norm_names["q"], (self.QD,), init="norm"))
+            if self.own_kv:
+                s.append(TensorSpec(self.row_norm_names["k"], (self.KD,), init="norm"))
+        if self.head_gate_name:
+            s.append(TensorSpec(self.head_gate_name + self.wsuf, (self.H, self.E)))
         if self.v_mix_name:
             s.append(TensorSpec(self.v_mix_name, (), init="half"))       # the first layer's is stored too, and unused
         if self.sink_name:
@@ -203,7 +230,14 @@ class PagedAttention(OutputProduct, Mixer):
 
     def bind(self, tensors, run_dtype, device):
         # q, k and v rows go straight into the one matrix the product reads, a tensor at a time
-        self.w_qkv = fused_rows(tensors, [self.names[x] + self.wsuf for x, _ in self._projections()], device)
+        rows = [self.names[x] + self.wsuf for x, _ in self._projections()]
+        if self.head_gate_name:
+            rows.append(self.head_gate_name + self.wsuf)
+        self.w_qkv = fused_rows(tensors, rows, device)
+        if self.row_norm:
+            self.w_qkv = pad_rows(self.w_qkv)
+            self.norm_w = tuple(tensors[self.row_norm_names[x]].to(torch.float32).contiguous() if x == "q" or self.own_kv else None
+                                for x in ("q", "k"))
         if self.qkv_bias:
             self.b_qkv = fused_rows(tensors, [self.names[x] + self.bsuf for x, _ in self._projections()], device)
         self.w_o = tensors[self.names["o"] + self.wsuf].contiguous()
@@ -241,8 +275,46 @@ class PagedAttention(OutputProduct, Mixer):
         gate = self.w_gate.numel() if self.w_gate is not None else 0
         return 2.0 * T * (self.w_qkv.numel() + self.w_o.numel() + gate) + 2.0 * (self.QD + self.OD) * seen
 
+    @property
+    def operand_width(self):
+        """Width of the output product's operand where :meth:`operand` makes it (layers with a gate per head), else None."""
+        return self.OD if self.head_gate_name else None
+
+    def operand(self, ctx, xn, cache, state, write_cache, out):
+        """The output product's operand into ``out`` [T, OD], which may be a column slice of a wider array."""
+        att, gates = self._attend_row_norm(ctx, xn, cache, write_cache)
+        with kernels.phase("attn"):
+            kernels.head_gate(att, gates, out, self.H, self.dv)
+        return out
+
+    def _attend_row_norm(self, ctx, xn, cache, write_cache):
+        """Heads' outputs before the gate, and the gates (None: no gate)."""
+        if write_cache and not self.own_kv:
+            raise ValueError("a layer without key and value projections must read another schedule entry's cache")
+        T, G, meta = xn.shape[0], self.G if self.own_kv else 0, ctx.group_meta(cache.group)
+        q = ctx.buf("attn_q", (T, self.QD), xn.dtype)
+        gates = ctx.buf("attn_head_gates", (T, self.H), torch.float32) if self.head_gate_name else None
+        with kernels.phase("qkv"):
+            kernels.linear_row_norm_kv(xn, self.w_qkv, ctx.buf("attn_qkv32", (T, self.w_qkv.shape[0]), torch.float32), *self.norm_w,
+                                       self.qk_norm_eps, meta.slots if write_cache else None, q, cache.k, cache.v, gates, self.H, G,
+                                       self.d, self.dv)
+        return self._softmax_attention(ctx, q, cache, meta), gates
+
+    def _softmax_attention(self, ctx, q, cache, meta):
+        att = ctx.buf("attn_out", (q.shape[0], self.OD), q.dtype)
+        with kernels.phase("attn"):
+            kernels.paged_attention(q, cache.k, None if self.values_are_keys else cache.v, meta, ctx, self.H, self.G, self.d,
+                                    self.mask, self.scale, att, tiles=ctx.arrays(self.step_arrays_key()), dv=self.dv,
+                                    values_in_keys=self.values_are_keys, sinks=self.sinks, zero_sink=self.sink == "zero",
+                                    slopes=self.slopes, head_scales=self.head_scales, softcap=self.softcap)
+        return att
+
     def _attend(self, ctx, xn, cache, write_cache):
         T = xn.shape[0]
+        if self.head_gate_name:
+            return self.operand(ctx, xn, cache, None, write_cache, ctx.buf("attn_gated", (T, self.OD), xn.dtype))
+        if self.row_norm:
+            return self._attend_row_norm(ctx, xn, cache, write_cache)[0]
         q = ctx.buf("attn_q", (T, self.QD), xn.dtype)
         meta = ctx.group_meta(cache.group)
         cos_sin = self.rotary.cos_sin if self.rotary is not None else None
@@ -268,12 +340,7 @@ class PagedAttention(OutputProduct, Mixer):
             with kernels.phase("qkv"):
                 kernels.linear_rope_kv(xn, self.w_qkv, self.b_qkv, qkv, cos_sin, n_rot, ctx.positions,
                                        meta.slots if write_cache else None, q, cache.k, cache.v, self.H, self.G, self.d)
-        att = ctx.buf("attn_out", (T, self.OD), xn.dtype)
-        with kernels.phase("attn"):
-            kernels.paged_attention(q, cache.k, None if self.values_are_keys else cache.v, meta, ctx, self.H, self.G, self.d,
-                                    self.mask, self.scale, att, tiles=ctx.arrays(self.step_arrays_key()), dv=self.dv,
-                                    values_in_keys=self.values_are_keys, sinks=self.sinks, zero_sink=self.sink == "zero",
-                                    slopes=self.slopes, head_scales=self.head_scales, softcap=self.softcap)
+        att = self._softmax_attention(ctx, q, cache, meta)
         if self.w_gate is not None:
             # the gate reads the mixer's input as the projections do; its sums stay float32 up to the sigmoid
             with kernels.phase("qkv"):

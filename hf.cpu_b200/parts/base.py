@@ -150,6 +150,9 @@ class Mixer(Part):
 
     # Optional: ``forward_then_norm(ctx, xn, residual, cache, state, write_cache, norm, out) -> bool`` does the same
     # and, if it returns True, has also written ``out = norm(residual)`` (the block then skips that norm).
+    # Optional: ``operand_width`` (not None) and ``operand(ctx, xn, cache, state, write_cache, out)``: writes the operand of
+    # the mixer's output product (``w_o``, ``b_o``) into ``out`` [T, operand_width], which may be a column slice of a wider
+    # array, and leaves the product to the caller.
 
 
 class FeedForward(Part):
@@ -157,7 +160,8 @@ class FeedForward(Part):
         """Token-wise transform of ``xn`` added into the float32 ``residual``."""
         raise NotImplementedError
 
-    # Optional: ``forward_then_norm(ctx, xn, residual, norm, out) -> bool``, as for mixers.
+    # Optional: ``forward_then_norm(ctx, xn, residual, norm, out) -> bool``, and ``operand_width`` with ``operand(ctx, xn, out)``
+    # (the product being ``w_down``, ``b_down``), as for mixers.
 
 
 class Block(Part):
@@ -165,6 +169,10 @@ class Block(Part):
         """Per-request state of the block itself (beside its mixer's), handed to ``forward`` as ``block_state``; one per
         schedule entry."""
         return None
+
+    def join_outputs(self, mixer: Mixer, ffn: Optional[FeedForward]) -> None:
+        """Called once when the layer's parts have their weights: a block whose sublayers read the same input may lay their
+        output products together."""
 
     def forward(self, ctx, x: torch.Tensor, norm1: Norm, mixer: Mixer, norm2: Norm, ffn: FeedForward,
                 cache, state, write_cache: bool, xn_ready: Optional[torch.Tensor] = None,

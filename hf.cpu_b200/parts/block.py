@@ -1,7 +1,7 @@
 """Residual arrangements.  Pre-norm: ``x += mixer(norm1(x)); x += ffn(norm2(x))`` (src/model.c:580-623); with a token
 shift, the mixer reads ``h_t + (h_(t-1) - h_t) * mu`` instead of ``h_t = norm1(x_t)``.
 Norm on both sides of each sublayer: ``x += post1(mixer(norm1(x))); x += post2(ffn(norm2(x)))``, where a layer may
-have no feed-forward at all.  Hyper-connections: the stream is kept in several copies; a sublayer reads a weighted
+have no feed-forward at all.  Parallel: ``x += mixer(h) + ffn(h)`` with one norm, ``h = norm1(x)``.  Hyper-connections: the stream is kept in several copies; a sublayer reads a weighted
 sum of them, and its output is written back into every copy while the copies are mixed among themselves."""
 from __future__ import annotations
 
@@ -135,6 +135,64 @@ class SandwichResidual(Block):
         return nxt if feed_forward(xn2, next_norm, nxt) else None
 
 
+class ParallelResidual(Block):
+    """``x += mixer(h) + ffn(h)``, ``h = norm1(x)``: both sublayers read the same normed input, there is no second norm, and a
+    layer may have no feed-forward.  Where both sublayers offer the operand of their last product, the two operands lie
+    side by side in one buffer and ONE product over the joined inner dimension ([W_o | W_down] [att; hidden]) ends the
+    layer: one pass over the stream, one sum in float32, the following norm in its tail."""
+    graph_safe = True
+
+    def __init__(self, **_):
+        self.w_out = self.b_out = None
+        self.widths = None                    # (mixer's, feed-forward's) columns of the joined operand
+
+    def join_outputs(self, mixer, ffn):
+        m, f = getattr(mixer, "operand_width", None), getattr(ffn, "operand_width", None)
+        if not m or not f:
+            return
+        if mixer.w_o.dtype == torch.bfloat16 and (m % 8 or f % 8):
+            return                            # the tensor-core product wants 16-byte rows and operands
+        self.w_out = torch.cat([mixer.w_o, ffn.w_down], 1).contiguous()
+        mixer.w_o, ffn.w_down = self.w_out[:, :m], self.w_out[:, m:]
+        b = [x for x in (getattr(mixer, "b_o", None), getattr(ffn, "b_down", None)) if x is not None]
+        self.b_out = b[0] if len(b) == 1 else (b[0].float() + b[1].float() if b else None)
+        self.widths = (m, f)
+
+    def forward(self, ctx, x, norm1, mixer, norm2, ffn, cache, state, write_cache, xn_ready=None, next_norm=None):
+        xn = xn_ready
+        if xn is None:
+            xn = ctx.buf("block_xn", x.shape, ctx.run_dtype)
+            norm1.forward(x, xn)
+        nxt = ctx.buf("block_xn", x.shape, ctx.run_dtype) if next_norm is not None else None     # (xn has been read by the time it is written)
+        if self.widths is not None:
+            m, f = self.widths
+            both = ctx.buf("block_operand", (x.shape[0], m + f), ctx.run_dtype)
+            mixer.operand(ctx, xn, cache, state, write_cache, both[:, :m])
+            ffn.operand(ctx, xn, both[:, m:])
+            args = next_norm.fused_args() if next_norm is not None else None
+            with kernels.phase("down"):
+                if args is None:
+                    kernels.linear(both, self.w_out, self.b_out, x, accumulate=True)
+                else:
+                    kernels.linear_residual_norm(both, self.w_out, self.b_out, x, args[0], args[1], nxt, **(args[2] if len(args) > 2 else {}))
+            if next_norm is not None and args is None:
+                next_norm.forward(x, nxt)
+            return nxt
+        last = None                           # what ends the layer, and may take the following norm along
+        if ffn is None:
+            fused = getattr(mixer, "forward_then_norm", None) if next_norm is not None else None
+            last = (lambda: fused(ctx, xn, x, cache, state, write_cache, next_norm, nxt)) if fused else \
+                (lambda: mixer.forward(ctx, xn, x, cache, state, write_cache))
+        else:
+            mixer.forward(ctx, xn, x, cache, state, write_cache)
+            fused = getattr(ffn, "forward_then_norm", None) if next_norm is not None else None
+            last = (lambda: fused(ctx, xn, x, next_norm, nxt)) if fused else (lambda: ffn.forward(ctx, xn, x))
+        done = last()
+        if next_norm is not None and not (fused and done):
+            next_norm.forward(x, nxt)
+        return nxt
+
+
 class HyperResidual(Block):
     """The stream in ``streams`` copies x_1 .. x_S ([T, S * E] float32, a token's copies side by side).  Sublayer q (1: the
     mixer, 2: the feed-forward) with its tensors ``<prefix>.hc<q>.{in [S], mix [S, S], out [S]}`` and, with ``layer_scale``,
@@ -238,5 +296,6 @@ class HyperResidual(Block):
 
 
 register_part("block", "hyper_residual", HyperResidual)
+register_part("block", "parallel_residual", ParallelResidual)
 register_part("block", "prenorm_residual", PreNormResidual)
 register_part("block", "sandwich_residual", SandwichResidual)

@@ -77,10 +77,11 @@ class HashedPairEmbedding(Embedding):
 class LinearHead(Part):
     graph_safe = True
 
-    def __init__(self, vocab_size: int, hidden_size: int, tensor: str, tied_to=None, scale: float = 1.0, **_):
+    def __init__(self, vocab_size: int, hidden_size: int, tensor: str, tied_to=None, scale: float = 1.0, softcap: float = 0.0, **_):
         self.vocab_size, self.hidden_size = int(vocab_size), int(hidden_size)
         self.tensor, self.tied_to = tensor, tied_to
         self.scale = float(scale)               # logits = (head . x) * scale
+        self.softcap = float(softcap or 0.0)    # ... then softcap * tanh(logits / softcap), 0: no cap
         self.weight = None
 
     def tensor_specs(self):
@@ -105,6 +106,8 @@ class LinearHead(Part):
             kernels.linear(xn, self.weight, None, logits, accumulate=False)
             if self.scale != 1.0:
                 kernels.scale_(logits, self.scale)
+            if self.softcap:
+                kernels.softcap_(logits, self.softcap)
         return logits
 
 

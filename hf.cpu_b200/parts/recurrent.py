@@ -1,7 +1,8 @@
 """Mixers that keep state of fixed size per request instead of keys and values per token: a matrix per head (the two
-gated linear recurrences below) or a vector (``mingru``, at the end).
+gated linear recurrences below, whose decay is a vector per head, and ``retention`` and ``mamba2``, whose decay is one
+number per head) or a vector (``mingru``).
 
-Both run the gated linear recurrence per head, with a state S [d, dv] that starts at zero for a new request, lives in
+The first two run the gated linear recurrence per head, with a state S [d, dv] that starts at zero for a new request, lives in
 float32 in the request's state slot and is carried from token to token:
 
 * ``gated_linear_attention``: ``S <- diag(a) S + k v^T``, ``o = S^T q``, with ``q = Wq h * d^(-1/2)``, ``k = Wk h``,
@@ -25,7 +26,7 @@ import torch
 
 from .. import kernels
 from ..config.base import UnsupportedError
-from ..weights.loader import TensorSpec, fused_rows
+from ..weights.loader import TensorSpec, fused_rows, pad_rows
 from .attention import OutputProduct
 from .base import Mixer, StateSpec, register_part
 
@@ -266,6 +267,177 @@ class MinGru(_Recurrent):
         return att
 
 
+class _ScalarDecay(_Recurrent):
+    """What the two mixers with one decay per head and token share.  Per head, S [d, dv] from zero in float32:
+
+        S_t = a_t S_(t-1) + c_t k_t u_t^T,   o_t = S_t^T q_t (+ D u_t)
+
+    One product makes everything that is read from the input, its float32 sums pass through a kernel that makes the
+    recurrence's operands (heads padded with zeros to a multiple of 16), the recurrence runs as a walk along the tokens or,
+    in steps with longer portions of the bfloat16 run, in chunks (``kernels.decay_scan``), and one kernel norms and gates
+    its output into the output product's operand.  ``operand`` writes that operand wherever it is asked to, so that a
+    block may lay it beside a feed-forward's and end both in one product."""
+    ARRAYS = ("decay_chunks",)
+
+    def step_arrays_key(self):
+        return self.ARRAYS
+
+    def step_arrays(self, batch):
+        return kernels.decay_chunk_arrays(batch.q_lens)
+
+    @property
+    def n_matrix(self):
+        return self.H * kernels.padded_head(self.dv) * kernels.padded_head(self.d)
+
+    def _matrix(self, state):
+        return state[:, :self.n_matrix].view(state.shape[0], self.H, kernels.padded_head(self.dv), kernels.padded_head(self.d))
+
+    @property
+    def operand_width(self):
+        """Width of the output product's operand (what :meth:`operand` writes)."""
+        return self.H * self.dv
+
+    def weight_bytes(self):
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o))
+
+    def flops(self, q_lens, kv_lens):
+        T = sum(q_lens)
+        return 2.0 * T * (self.w_in.numel() + self.w_o.numel()) + 5.0 * T * self.H * self.d * self.dv
+
+    def _operands(self, ctx, T, Hq, dtype):
+        dp, dvp = kernels.padded_head(self.d), kernels.padded_head(self.dv)
+        return (ctx.buf("decay_q", (T, Hq * dp), dtype), ctx.buf("decay_k", (T, Hq * dp), dtype),
+                ctx.buf("decay_u", (T, self.H * dvp), dtype))
+
+    def _attend(self, ctx, xn, cache, write_cache, state):
+        return self.operand(ctx, xn, cache, state, write_cache, ctx.buf("rec_att", (xn.shape[0], self.operand_width), xn.dtype))
+
+
+class Retention(_ScalarDecay):
+    """Linear attention with a fixed decay per head and no softmax: q = Wq h and k = Wk h rotated (dimension i with i +
+    n_rot/2 of the leading n_rot), k times ``head_dim^(-1/2)``, u = v = Wv h, ``a`` the head's entry of ``decay``; every
+    head's o is divided by its root mean square (no weight), then multiplied by silu(Wg h), then ``Wo``."""
+
+    def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decay, norm_eps: float, prefix: str,
+                 position=None, positions=None, names=None, **_):
+        self.E, self.H, self.d, self.dv = int(hidden_size), int(num_heads), int(head_dim), int(v_head_dim)
+        self.eps, self.prefix = float(norm_eps), prefix
+        self.decay = [float(a) for a in decay]
+        if len(self.decay) != self.H or not all(0.0 <= a <= 1.0 for a in self.decay):
+            raise UnsupportedError(f"retention: one decay between 0 and 1 for each of the {self.H} heads")
+        if kernels.padded_head(self.d) > kernels.SCAN_MAX_HEAD:
+            raise UnsupportedError(f"retention: key heads above {kernels.SCAN_MAX_HEAD} are not supported")
+        self.rotary = (positions or {}).get(position) if position else None
+        if position and self.rotary is None:
+            raise UnsupportedError(f"retention names position encoding '{position}', which the plan does not define")
+        if self.rotary is not None and getattr(self.rotary, "pairing", "half") != "half":
+            raise UnsupportedError("retention: the rotation pairs dimension i with i + n_rot/2")
+        n = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
+        n.update(names or {})
+        self.nm = n
+        self.w_in = self.w_o = self.log_decay = None
+
+    def state_spec(self):
+        return StateSpec((self.n_matrix,))
+
+    def tensor_specs(self):
+        KD, VD = self.H * self.d, self.H * self.dv
+        return [TensorSpec(self._t("q"), (KD, self.E)), TensorSpec(self._t("k"), (KD, self.E)), TensorSpec(self._t("v"), (VD, self.E)),
+                TensorSpec(self._t("g"), (VD, self.E)), TensorSpec(self._t("o"), (self.E, VD))]
+
+    def bind(self, tensors, run_dtype, device):
+        self.w_in = pad_rows(fused_rows(tensors, [self._t(x) for x in ("q", "k", "v", "g")], device))
+        self.w_o = tensors[self._t("o")].contiguous()
+        # the logarithm in float64 from the configuration's numbers; a decay of zero as one that leaves nothing
+        la = torch.tensor(self.decay, dtype=torch.float64).log().clamp_(min=-1e4)
+        self.log_decay = la.to(torch.float32).to(device)
+
+    def operand(self, ctx, xn, cache, state, write_cache, out):
+        T = xn.shape[0]
+        KD, VD, C = self.H * self.d, self.H * self.dv, self.w_in.shape[0]
+        q, k, u = self._operands(ctx, T, self.H, xn.dtype)
+        cos_sin, n_rot = (self.rotary.cos_sin, self.rotary.n_rot) if self.rotary is not None else (None, 0)
+        with kernels.phase("qkv"):
+            row, splits = kernels.product_sums(xn, self.w_in, ctx.buf("rec_in", (T, C), torch.float32))
+            kernels.rotate_heads(row, splits, C, cos_sin, n_rot, ctx.positions, self.d ** -0.5, q, k, u, self.H, self.d, self.dv)
+        o = ctx.buf("rec_o", (T, VD), torch.float32)
+        with kernels.phase("attn"):
+            kernels.decay_scan(q, k, u, self.log_decay, None, None, self._matrix(state), ctx, o, self.H, self.H, self.d, self.dv,
+                               chunks=ctx.arrays(self.ARRAYS))
+            kernels.part_norm_gate(o, self.H, self.eps, row, splits, C, 2 * KD + VD, None, False, out)
+        return out
+
+
+class Mamba2(_ScalarDecay):
+    """Mamba-2's state-space recurrence (state-space duality, Dao and Gu 2024).  One product gives [z | x | B | C | dt]; x, B
+    and C pass a causal convolution per channel with a bias and silu; step = softplus(dt + dt_bias); per head (value head h
+    reads group ``h // (H / groups)``) ``a = exp(-exp(A_log) step)``, c = step, k = B, q = C, u = x, plus ``D x``; the heads'
+    outputs times silu(z), rms-normed in ``norm_groups`` equal parts with a weight, then ``Wo``.  The convolution's last ``taps -
+    1`` inputs are part of the request's state."""
+
+    def __init__(self, hidden_size: int, num_heads: int, v_head_dim: int, state_size: int, groups: int, conv_taps: int, norm_groups: int,
+                 norm_eps: float, prefix: str, names=None, **_):
+        self.E, self.H, self.dv, self.d, self.G = int(hidden_size), int(num_heads), int(v_head_dim), int(state_size), int(groups)
+        self.taps, self.norm_groups, self.eps, self.prefix = int(conv_taps), int(norm_groups), float(norm_eps), prefix
+        if self.H % self.G:
+            raise UnsupportedError(f"mamba2: {self.H} heads over {self.G} groups")
+        if (self.H * self.dv) % self.norm_groups:
+            raise UnsupportedError(f"mamba2: {self.H * self.dv} channels in {self.norm_groups} norm groups")
+        if not 1 <= self.taps <= kernels.CONV_MAX_TAPS:
+            raise UnsupportedError(f"mamba2: {self.taps} convolution taps (1 to {kernels.CONV_MAX_TAPS})")
+        if kernels.padded_head(self.d) > kernels.SCAN_MAX_HEAD:
+            raise UnsupportedError(f"mamba2: states above {kernels.SCAN_MAX_HEAD} are not supported")
+        n = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "A": "A_log", "D": "D", "norm": "norm", "o": "o"}
+        n.update(names or {})
+        self.nm = n
+        self.w_in = self.w_o = self.w_conv = self.b_conv = self.dt_bias = self.rate = self.skip = self.norm_w = None
+
+    @property
+    def C(self):
+        """Channels of the convolution: x, B and C side by side."""
+        return self.H * self.dv + 2 * self.G * self.d
+
+    def state_spec(self):
+        n = self.n_matrix + max(self.taps - 1, 1) * self.C
+        return StateSpec(((n + 3) // 4 * 4,))
+
+    def tensor_specs(self):
+        VD = self.H * self.dv
+        return [TensorSpec(self._t("in"), (VD + self.C + self.H, self.E)), TensorSpec(self._t("conv"), (self.C, self.taps)),
+                TensorSpec(self._t("conv_bias"), (self.C,)), TensorSpec(self._t("dt_bias"), (self.H,)), TensorSpec(self._t("A"), (self.H,)),
+                TensorSpec(self._t("D"), (self.H,), init="norm"), TensorSpec(self._t("norm"), (VD,), init="norm"),
+                TensorSpec(self._t("o"), (self.E, VD))]
+
+    def bind(self, tensors, run_dtype, device):
+        self.w_in = pad_rows(tensors[self._t("in")])
+        self.w_o = tensors[self._t("o")].contiguous()
+        self.w_conv, self.b_conv = tensors[self._t("conv")].contiguous(), tensors[self._t("conv_bias")].contiguous()
+        self.dt_bias = tensors[self._t("dt_bias")].contiguous()
+        self.rate = torch.exp(tensors[self._t("A")].to(torch.float32)).contiguous()
+        self.skip = tensors[self._t("D")].to(torch.float32).contiguous()
+        self.norm_w = tensors[self._t("norm")].to(torch.float32).contiguous()
+
+    def operand(self, ctx, xn, cache, state, write_cache, out):
+        T = xn.shape[0]
+        VD, C = self.H * self.dv, self.w_in.shape[0]
+        q, k, u = self._operands(ctx, T, self.G, xn.dtype)
+        step, la = ctx.buf("decay_step", (T, self.H), torch.float32), ctx.buf("decay_la", (T, self.H), torch.float32)
+        K = max(self.taps - 1, 1)
+        carried = state[:, self.n_matrix:self.n_matrix + K * self.C].view(state.shape[0], K, self.C)
+        with kernels.phase("qkv"):
+            row, splits = kernels.product_sums(xn, self.w_in, ctx.buf("rec_in", (T, C), torch.float32))
+            kernels.state_space_operands(row, splits, C, self.w_conv, self.b_conv, self.dt_bias, self.rate, carried, ctx, q, k, u, step, la,
+                                         self.H, self.G, self.d, self.dv)
+        o = ctx.buf("rec_o", (T, VD), torch.float32)
+        with kernels.phase("attn"):
+            kernels.decay_scan(q, k, u, la, step, self.skip, self._matrix(state), ctx, o, self.H, self.G, self.d, self.dv,
+                               chunks=ctx.arrays(self.ARRAYS))
+            kernels.part_norm_gate(o, self.norm_groups, self.eps, row, splits, C, 0, self.norm_w, True, out)
+        return out
+
+
+register_part("mixer", "retention", Retention)
+register_part("mixer", "mamba2", Mamba2)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "mingru", MinGru)
 register_part("mixer", "gated_delta_rule", GatedDeltaRule)

@@ -203,6 +203,13 @@ def fused_rows(tensors, names: Sequence[str], device: torch.device, interleave: 
     return out
 
 
+def pad_rows(w: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """The matrix with rows of zeros behind it up to a multiple of ``multiple`` rows, so that what reads a product's rows
+    finds aligned vectors."""
+    short = -w.shape[0] % multiple
+    return torch.cat([w, w.new_zeros((short,) + tuple(w.shape[1:]))]) if short else w.contiguous()
+
+
 class _Staging:
     """Two pinned buffers through which file bytes go to the device: one is filled from the file mapping while
     the copy out of the other is in flight."""

@@ -238,9 +238,16 @@ class EmuBackend:
             return torch.relu(z) ** 2
         return z
 
-    def linear_glu(self, a, w, gu_buf, out, act):
+    def linear_glu(self, a, w, gu_buf, out, act, bias=None, clamp=None):
         self.linear(a, w, None, gu_buf, False)
+        if bias is not None:
+            gu_buf = gu_buf.float() + bias.float()
         g, u = gu_buf[:, 0::2].float(), gu_buf[:, 1::2].float()
+        if clamp is not None:
+            limit, alpha, offset = clamp
+            g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+            out.copy_((g * torch.sigmoid(alpha * g) * (u + offset)).to(out.dtype))
+            return
         out.copy_((self._activate(g, act) * u).to(out.dtype))
 
     def linear_act(self, a, w, out, act):
@@ -248,6 +255,9 @@ class EmuBackend:
 
     def scale_(self, x, s):
         x.mul_(s)
+
+    def softcap_(self, x, cap):
+        x.copy_(cap * torch.tanh(x / cap))
 
     def moe_route(self, h, w, b, top, ids, weights, logits):
         z = h.float() @ w.float().T
@@ -406,6 +416,95 @@ class EmuBackend:
                 S = (1.0 - z[t]) * S + z[t] * cand[t]
                 out[t] = (S * g[t] * torch.sigmoid(g[t])).to(out.dtype)
             state[slots[s]] = S
+
+    # ---- recurrences with one decay per head and token
+    @staticmethod
+    def _pad_heads(x, dst, heads):
+        """x [T, heads, n] into dst [T, heads * padded n] with zeros behind every head."""
+        d = dst.view(dst.shape[0], heads, -1)
+        d.zero_()
+        d[..., :x.shape[-1]] = x.to(dst.dtype)
+
+    def rotate_heads(self, src, splits, row, cos_sin, n_rot, positions, k_scale, q, k, u, H, d, dv):
+        T = q.shape[0]
+        r = src.reshape(-1)[:splits * T * row].view(splits, T, row).sum(0)
+        qk = r[:, :2 * H * d].view(T, 2 * H, d).clone()
+        if n_rot:
+            half = n_rot // 2
+            cs = cos_sin[positions.long()]
+            c, s = cs[:, None, :, 0], cs[:, None, :, 1]
+            x, y = qk[..., :half].clone(), qk[..., half:n_rot].clone()
+            qk[..., :half], qk[..., half:n_rot] = x * c - y * s, y * c + x * s
+        self._pad_heads(qk[:, :H], q, H)
+        self._pad_heads(qk[:, H:] * k_scale, k, H)
+        self._pad_heads(r[:, 2 * H * d:2 * H * d + H * dv].view(T, H, dv), u, H)
+
+    def state_space_operands(self, src, splits, row, conv_w, conv_b, dt_bias, rate, carried, ctx, q, k, u, step, la, H, G, d, dv):
+        T, inner, taps = q.shape[0], H * dv, conv_w.shape[1]
+        C, K = inner + 2 * G * d, taps - 1
+        r = src.reshape(-1)[:splits * T * row].view(splits, T, row).sum(0)
+        x = r[:, inner:inner + C]
+        y = torch.zeros(T, C, device=src.device)
+        cu, slots = ctx.cu_tokens.tolist(), ctx.seq_slots.tolist()
+        for s in range(len(slots)):
+            seen = torch.cat([carried[slots[s]][:K], x[cu[s]:cu[s + 1]]])
+            for t in range(cu[s + 1] - cu[s]):
+                y[cu[s] + t] = conv_b.float() + (seen[t:t + taps] * conv_w.float().T).sum(0)
+            if K:
+                carried[slots[s]] = seen[-K:]
+        y = y * torch.sigmoid(y)
+        self._pad_heads(y[:, :inner].view(T, H, dv), u, H)
+        self._pad_heads(y[:, inner:inner + G * d].view(T, G, d), k, G)
+        self._pad_heads(y[:, inner + G * d:].view(T, G, d), q, G)
+        step.copy_(torch.nn.functional.softplus(r[:, inner + C:inner + C + H] + dt_bias.float()))
+        la.copy_(-rate * step)
+
+    def decay_scan(self, q, k, u, la, step, skip, state, ctx, o, H, Hq, d, dv, chunks):
+        T = q.shape[0]
+        rep = H // Hq
+        qh = q.float().view(T, Hq, -1).repeat_interleave(rep, 1)
+        kh = k.float().view(T, Hq, -1).repeat_interleave(rep, 1)
+        uh = u.float().view(T, H, -1)
+        a = torch.exp(la).expand(T, H)
+        cu, slots = ctx.cu_tokens.tolist(), ctx.seq_slots.tolist()
+        for s in range(len(slots)):
+            S = state[slots[s]].clone()                                        # [H, dvp, dp]
+            for t in range(cu[s], cu[s + 1]):
+                ut = uh[t] if step is None else uh[t] * step[t][:, None]
+                S = a[t][:, None, None] * S + ut[:, :, None] * kh[t][:, None, :]
+                y = (S * qh[t][:, None, :]).sum(-1)
+                if skip is not None:
+                    y = y + skip[:, None] * uh[t]
+                o[t] = y[:, :dv].reshape(-1)
+            state[slots[s]] = S
+
+    def part_norm_gate(self, o, parts, eps, g, g_splits, g_stride, g_col0, w, gate_first, out):
+        T, C = o.shape
+        z = g.reshape(-1)[:g_splits * T * g_stride].view(g_splits, T, g_stride).sum(0)[:, g_col0:g_col0 + C]
+        gate = z * torch.sigmoid(z)
+        y = o * gate if gate_first else o
+        p = y.view(T, parts, -1)
+        y = (p / torch.sqrt((p * p).mean(-1, keepdim=True) + eps)).reshape(T, C)
+        if w is not None:
+            y = y * w
+        out.copy_((y if gate_first else y * gate).to(out.dtype))
+
+    # ---- attention normed over the whole projection, head gates
+    def linear_row_norm_kv(self, a, w, buf, q_w, k_w, eps, slots, q_out, k_cache, v_cache, gate_out, H, G, d, dv):
+        r = a.float() @ w.float().T
+        QD, KD, VD = H * d, G * d, G * dv
+        norm = lambda x, wt: x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * wt
+        q_out.copy_(norm(r[:, :QD], q_w).to(q_out.dtype))
+        if G and slots is not None:
+            k_cache.view(-1, KD)[slots.long()] = norm(r[:, QD:QD + KD], k_w).to(k_cache.dtype)
+            v_cache.view(-1, VD)[slots.long()] = r[:, QD + KD:QD + KD + VD].to(v_cache.dtype)
+        if gate_out is not None:
+            n = gate_out.shape[1]
+            gate_out.copy_(torch.sigmoid(r[:, QD + KD + VD:QD + KD + VD + n]))
+
+    def head_gate(self, a, gate, out, H, dv):
+        T = a.shape[0]
+        out.copy_((a.float().view(T, H, dv) * gate[:, :, None]).view(T, H * dv).to(out.dtype))
 
     def moe_group(self, ids, experts, order, tile_expert, tile_p0, tile_n, n_tiles, tile):
         MOE_TILE = tile
