@@ -343,10 +343,33 @@ def silupel_configs(z):
     return silupel, peludra
 
 
+# ---- `--compare tupalorn`: the Tupalorn design beside the Silupel design at equal layer sizes ------------------------
+# Nine layers in threes: Mamba-2 (twice the stream's width, value heads of 64, states of 128), retention, windowed
+# attention with a gate per head, the last of which reads the keys and values of the one before it; every layer parallel
+# with a clamped gated feed-forward.  The Silupel twin is that of `--compare silupel`: nine layer runs, the same attention
+# heads, a gated feed-forward of the same size.
+TUPALORN_SIZES = {n: dict(z, window=1024, rdim=128 if z["width"] > 1024 else 64) for n, z in SILUPEL_SIZES.items()}
+
+
+def tupalorn_configs(z):
+    m2 = dict(heads=2 * z["width"] // 64, vdim=64, state=128, groups=1, conv=4, norm_groups=1)
+    n = z["width"] // z["rdim"]
+    ret = dict(heads=n, dim=z["rdim"], vdim=z["rdim"], decay=[1.0 - 2.0 ** (-5.0 - 4.0 * i / n) for i in range(n)],
+               rot=dict(dims=z["rdim"], base=10000.0))
+    att = dict(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5, mask=dict(size=z["window"]))
+    kinds = (dict(type="mamba2", mixer=m2), dict(type="retention", mixer=ret), dict(type="attention", mixer=att))
+    layers = [dict(kinds[i % 3], mlp=dict(kind="dense", ff=z["ff"], limit=7.0)) for i in range(9)]
+    layers[8] = dict(layers[8], mixer=dict(att, kv_from=5))
+    tupalorn = dict(architecture="Tupalorn", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), logit_softcap=30.0,
+                    max_positions=8192, layers=layers)
+    return tupalorn, silupel_configs(z)[0]
+
+
 COMPARISONS = {"manapel": (COMPARE_SIZES, compare_configs), "peludra": (PELUDRA_SIZES, peludra_configs),
-               "mokisun": (MOKISUN_SIZES, mokisun_configs), "silupel": (SILUPEL_SIZES, silupel_configs)}
+               "mokisun": (MOKISUN_SIZES, mokisun_configs), "silupel": (SILUPEL_SIZES, silupel_configs),
+               "tupalorn": (TUPALORN_SIZES, tupalorn_configs)}
 # the design each comparison stands beside
-TWINS = {"manapel": "qwen2", "peludra": "qwen2", "mokisun": "manapel", "silupel": "peludra"}
+TWINS = {"manapel": "qwen2", "peludra": "qwen2", "mokisun": "manapel", "silupel": "peludra", "tupalorn": "silupel"}
 
 
 def phase_work(model, q_len, ctx_len, batch):
@@ -405,8 +428,20 @@ def phase_work(model, q_len, ctx_len, batch):
         add("attn", 12.0 * T * m.W, 4 * (T * 3 * m.W + 2 * batch * m.W) + el * T * m.W)
         add("wo", 2.0 * T * m.w_o.numel(), el * (m.w_o.numel() + T * m.W) + 4 * T * m.E)
 
+    def scalar_decay(m):
+        # one product in front (float32 sums out, which the recurrence's operands are made from: read once, bfloat16 out); the
+        # recurrence reads its operands, reads and writes every request's state once and stores float32 rows, which the
+        # norm and gate pass reads with the gate's sums; its operations are counted for the walk, token by token
+        Hq = getattr(m, "G", m.H)
+        rows = T * (2 * Hq * m.d + m.H * m.dv)
+        add("qkv", 2.0 * T * m.w_in.numel(), el * (m.w_in.numel() + T * m.E) + 8 * T * m.w_in.shape[0] + el * rows)
+        add("attn", 5.0 * T * m.H * m.d * m.dv, el * rows + 8 * batch * m.n_matrix + (12 + el) * T * m.H * m.dv)
+        add("wo", 2.0 * T * m.w_o.numel(), el * (m.w_o.numel() + T * m.H * m.dv) + 4 * T * m.E)
+
     def mixer(m):
-        if hasattr(m, "branches"):
+        if hasattr(m, "n_matrix") and hasattr(m, "operand"):
+            scalar_decay(m)
+        elif hasattr(m, "branches"):
             for b in m.branches:
                 mixer(b)
         elif hasattr(m, "b_z"):
@@ -418,7 +453,12 @@ def phase_work(model, q_len, ctx_len, batch):
     for e in model.plan.schedule:
         L = model.layers[e.layer]
         f = L.ffn
+        before = list(work["wo"])
         mixer(L.mixer)
+        if getattr(L.block, "widths", None) is not None:
+            # one product ends both sublayers; its time is the feed-forward's down phase
+            add("down", work["wo"][0] - before[0], work["wo"][1] - before[1] - 4 * T * f.E)
+            work["wo"] = before
         if hasattr(f, "w_up"):
             add("gate_up", 2.0 * T * f.w_up.numel(), el * (f.w_up.numel() + T * (f.E + f.F)))
             add("down", 2.0 * T * f.w_down.numel(), el * (f.w_down.numel() + T * f.F) + 4 * T * f.E)

@@ -40,6 +40,44 @@ __device__ __forceinline__ void store_any(void *p, int dt, size_t i, float v)
     else ((__nv_bfloat16 *)p)[i] = __float2bfloat16_rn(v);
 }
 
+// The sum of a value's `splits` planes, eight reads in flight.
+__device__ __forceinline__ float plane_sum(const float *p, int splits, size_t plane)
+{
+    float v = p[0];
+    for (int s = 1; s < splits; s += 8) {
+        float x[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) x[j] = s + j < splits ? p[(size_t)(s + j) * plane] : 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; j++) v += x[j];
+    }
+    return v;
+}
+__device__ __forceinline__ float2 plane_sum2(const float *p, int splits, size_t plane)
+{
+    float2 v = *(const float2 *)p;
+    for (int s = 1; s < splits; s += 8) {
+        float2 x[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) x[j] = s + j < splits ? *(const float2 *)(p + (size_t)(s + j) * plane) : make_float2(0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < 8; j++) { v.x += x[j].x; v.y += x[j].y; }
+    }
+    return v;
+}
+__device__ __forceinline__ float4 plane_sum4(const float *p, int splits, size_t plane)
+{
+    float4 v = *(const float4 *)p;
+    for (int s = 1; s < splits; s += 4) {
+        float4 x[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) x[j] = s + j < splits ? *(const float4 *)(p + (size_t)(s + j) * plane) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < 4; j++) { v.x += x[j].x; v.y += x[j].y; v.z += x[j].z; v.w += x[j].w; }
+    }
+    return v;
+}
+
 __device__ __forceinline__ float warp_sum(float v)
 {
 #pragma unroll

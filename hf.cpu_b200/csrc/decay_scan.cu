@@ -35,6 +35,8 @@ constexpr int DS_MAX_CHUNK_D = 256;   // largest padded key head of the chunk fo
 constexpr int DS_MAX_D = 512;         // ... and of the walk
 constexpr int DS_MAX_TAPS = 16;
 
+static bool aligned16(const void *p) { return ((uintptr_t)p & 15) == 0; }
+
 template <typename T> struct Pack4;
 template <> struct Pack4<float> {
     static __device__ __forceinline__ float4 load(const float *p) { return *(const float4 *)p; }
@@ -48,6 +50,17 @@ template <> struct Pack4<__nv_bfloat16> {
     }
 };
 
+// exp and z * sigmoid(z): from the special-function unit where the result is rounded to bfloat16 behind it, else CUDA's
+// full-accuracy functions.
+template <typename TO> __device__ __forceinline__ float silu_for(float z)
+{
+    if constexpr (sizeof(TO) == 4) return z / (1.0f + expf(-z));
+    else return __fdividef(z, 1.0f + __expf(-z));
+}
+
+__device__ __forceinline__ void store2(float *p, float a, float b) { *(float2 *)p = make_float2(a, b); }
+__device__ __forceinline__ void store2(__nv_bfloat16 *p, float a, float b) { *(__nv_bfloat162 *)p = __floats2bfloat162_rn(a, b); }
+
 // ---- operands of retention --------------------------------------------------------------------------------------
 // One warp per (token, head) of the rows [H query heads of d | H key heads of d | H value heads of dv | ...] (row_stride
 // floats, `splits` planes): rotation of the first n_rot dimensions of queries and keys (pairs i, i + n_rot/2), keys times
@@ -55,7 +68,8 @@ template <> struct Pack4<__nv_bfloat16> {
 template <typename TO>
 __global__ void __launch_bounds__(128)
 rotate_heads_kernel(const float *src, int splits, int row_stride, const float *cos_sin, int n_rot, int n_positions,
-                    const int32_t *positions, float k_scale, TO *q, TO *k, TO *u, int T, int H, int d, int dv, int dp, int dvp, int *err)
+                    const int32_t *positions, float k_scale, TO *q, TO *k, TO *u, int T, int H, int d, int dv, int dp, int dvp, int pairs,
+                    int *err)
 {
     pdl_entry();
     pdl_sync_small();
@@ -71,37 +85,61 @@ rotate_heads_kernel(const float *src, int splits, int row_stride, const float *c
         if (pos < 0 || pos >= n_positions) { if (lane == 0) atomicOr(err, HFB_ERR_POSITION); pos = 0; }
     }
     const float *cs = cos_sin + (size_t)pos * n_rot;
-    auto sum = [&](int c) {
-        float v = row[c];
-        for (int s = 1; s < splits; s++) v += row[(size_t)s * plane + c];
-        return v;
-    };
-#pragma unroll
+    const float *qr = row + h * d, *kr = qr + H * d, *vr = row + 2 * H * d + h * dv;
+    TO *qd = q + ((size_t)t * H + h) * dp, *kd = k + ((size_t)t * H + h) * dp, *ud = u + ((size_t)t * H + h) * dvp;
+    if (pairs) {
+        // two neighbouring dimensions a lane: everything of the head is even and aligned to two
+        for (int i = 2 * lane; i < half; i += 64) {
+            const float4 c = *(const float4 *)(cs + 2 * i);
+            const float2 qa = plane_sum2(qr + i, splits, plane), qb = plane_sum2(qr + i + half, splits, plane);
+            const float2 ka = plane_sum2(kr + i, splits, plane), kb = plane_sum2(kr + i + half, splits, plane);
+            float lo0, hi0, lo1, hi1;
+            rope_pair(qa.x, qb.x, c.x, c.y, lo0, hi0);
+            rope_pair(qa.y, qb.y, c.z, c.w, lo1, hi1);
+            store2(qd + i, lo0, lo1);
+            store2(qd + i + half, hi0, hi1);
+            rope_pair(ka.x, kb.x, c.x, c.y, lo0, hi0);
+            rope_pair(ka.y, kb.y, c.z, c.w, lo1, hi1);
+            store2(kd + i, lo0 * k_scale, lo1 * k_scale);
+            store2(kd + i + half, hi0 * k_scale, hi1 * k_scale);
+        }
+        for (int i = n_rot + 2 * lane; i < dp; i += 64) {
+            const float2 a = i < d ? plane_sum2(qr + i, splits, plane) : make_float2(0.f, 0.f);
+            const float2 b = i < d ? plane_sum2(kr + i, splits, plane) : make_float2(0.f, 0.f);
+            store2(qd + i, a.x, a.y);
+            store2(kd + i, b.x * k_scale, b.y * k_scale);
+        }
+        for (int i = 2 * lane; i < dvp; i += 64) {
+            const float2 a = i < dv ? plane_sum2(vr + i, splits, plane) : make_float2(0.f, 0.f);
+            store2(ud + i, a.x, a.y);
+        }
+        return;
+    }
+#pragma unroll 1
     for (int part = 0; part < 2; part++) {
-        const int c0 = (part * H + h) * d;
-        TO *dst = (part ? k : q) + ((size_t)t * H + h) * dp;
+        const float *p = part ? kr : qr;
+        TO *dst = part ? kd : qd;
         const float f = part ? k_scale : 1.0f;
         for (int i = lane; i < half; i += 32) {
             float lo, hi;
-            rope_pair(sum(c0 + i), sum(c0 + i + half), cs[2 * i], cs[2 * i + 1], lo, hi);
+            rope_pair(plane_sum(p + i, splits, plane), plane_sum(p + i + half, splits, plane), cs[2 * i], cs[2 * i + 1], lo, hi);
             dst[i] = from_f32<TO>(lo * f);
             dst[i + half] = from_f32<TO>(hi * f);
         }
-        for (int i = n_rot + lane; i < dp; i += 32) dst[i] = from_f32<TO>(i < d ? sum(c0 + i) * f : 0.f);
+        for (int i = n_rot + lane; i < dp; i += 32) dst[i] = from_f32<TO>(i < d ? plane_sum(p + i, splits, plane) * f : 0.f);
     }
-    const int c0 = 2 * H * d + h * dv;
-    TO *dst = u + ((size_t)t * H + h) * dvp;
-    for (int i = lane; i < dvp; i += 32) dst[i] = from_f32<TO>(i < dv ? sum(c0 + i) : 0.f);
+    for (int i = lane; i < dvp; i += 32) ud[i] = from_f32<TO>(i < dv ? plane_sum(vr + i, splits, plane) : 0.f);
 }
 
 // ---- operands of the state-space form ---------------------------------------------------------------------------
 // Rows (row_stride floats, `splits` planes): [z: H dv | x: H dv | B: G d | C: G d | dt: H | ...].  x, B and C pass a causal
-// convolution per channel (w [CC, taps], last column the current token's; bias [CC]) and silu: x to u, B to k, C to q.
-// step[t, h] = softplus(dt + dt_bias), la[t, h] = -rate[h] * step.  Blocks: `tt` tokens x 128 channels, a thread per channel
-// that slides a window of taps along the tokens; the last blocks in x make step and la.  Inputs before a request's first
+// convolution per channel (w [CC, taps], last column the current token's; bias [CC]) and silu: x to u, B to k, C to q.  A
+// thread takes V neighbouring channels.
+// step[t, h] = softplus(dt + dt_bias), la[t, h] = -rate[h] * step.  Blocks: `tt` tokens x 128 V channels, a thread
+// slides a window of taps along the tokens; the last blocks in x make step and la.  Inputs before a request's first
 // token of this step come from its slot, carried [taps - 1][CC] oldest first (zeros for a new request).  `single`: every
 // request brings one token, and the thread brings its channel of the slot up to date itself (else conv_carry does).
-template <int TAPS, typename TO>
+template <int TAPS, int V, typename TO>
 __global__ void __launch_bounds__(128)
 state_space_operands_kernel(const float *src, int splits, int row_stride, const void *w, int w_dt, const void *bias, int bias_dt, int taps,
                             const void *dt_bias, int dtb_dt, const float *rate, float *carried, size_t slot_stride,
@@ -112,7 +150,7 @@ state_space_operands_kernel(const float *src, int splits, int row_stride, const 
     pdl_entry();
     pdl_sync_small();
     const int inner = H * dv, CC = inner + 2 * G * d;
-    const int conv_blocks = (CC + 127) / 128;
+    const int conv_blocks = (CC + 128 * V - 1) / (128 * V);
     const size_t plane = (size_t)T * row_stride;
     const int tb = blockIdx.y * tt, te = min(T, tb + tt);
     if ((int)blockIdx.x >= conv_blocks) {
@@ -122,29 +160,30 @@ state_space_operands_kernel(const float *src, int splits, int row_stride, const 
 #pragma unroll 4
         for (int t = tb; t < te; t++) {
             const float *p = src + (size_t)t * row_stride + 2 * inner + 2 * G * d + h;
-            float z = p[0];
-            for (int s = 1; s < splits; s++) z += p[(size_t)s * plane];
-            z += b;
+            const float z = plane_sum(p, splits, plane) + b;
             const float v = z > 20.f ? z : log1pf(expf(z));
             step[(size_t)t * H + h] = v;
             la[(size_t)t * H + h] = -r * v;
         }
         return;
     }
-    const int ch = blockIdx.x * 128 + threadIdx.x;
-    if (ch >= CC) return;
     constexpr int W = TAPS ? TAPS : DS_MAX_TAPS;
+    const int ch = (blockIdx.x * 128 + threadIdx.x) * V;
+    if (ch >= CC) return;
     const int n_taps = TAPS ? TAPS : taps, K = n_taps - 1;
     // the window holds the last n_taps inputs in its last n_taps places; weights likewise
-    float wv[W], win[W];
+    float wv[V][W], win[V][W], b[V];
 #pragma unroll
-    for (int j = 0; j < W; j++) {
-        const int i = j - (W - n_taps);
-        wv[j] = i >= 0 ? load_any(w, w_dt, (size_t)ch * n_taps + i) : 0.f;
-        win[j] = 0.f;
+    for (int c = 0; c < V; c++) {
+#pragma unroll
+        for (int j = 0; j < W; j++) {
+            const int i = j - (W - n_taps);
+            wv[c][j] = i >= 0 ? load_any(w, w_dt, (size_t)(ch + c) * n_taps + i) : 0.f;
+            win[c][j] = 0.f;
+        }
+        b[c] = load_any(bias, bias_dt, ch + c);
     }
-    const float b = load_any(bias, bias_dt, ch);
-    // where this channel goes
+    // where this thread's channels go (V = 2: heads of even size, so both belong to one)
     TO *dst;
     size_t dst_stride;
     int pad = 0;                                     // zeros behind a head's last channel
@@ -152,19 +191,22 @@ state_space_operands_kernel(const float *src, int splits, int row_stride, const 
         const int h = ch / dv, i = ch % dv;
         dst = u + (size_t)h * dvp + i;
         dst_stride = (size_t)H * dvp;
-        if (i == dv - 1) pad = dvp - dv;
+        if (i + V == dv) pad = dvp - dv;
     } else {
         const int c = ch - inner, which = c / (G * d), g = c % (G * d) / d, i = c % d;
         dst = (which ? q : k) + (size_t)g * dp + i;
         dst_stride = (size_t)G * dp;
-        if (i == d - 1) pad = dp - d;
+        if (i + V == d) pad = dp - d;
     }
     const float *x = src + inner + ch;
-    auto input = [&](int t) {
-        const float *p = x + (size_t)t * row_stride;
-        float v = p[0];
-        for (int s = 1; s < splits; s++) v += p[(size_t)s * plane];
-        return v;
+    auto input = [&](int t, float *v) {
+        if constexpr (V == 2) {
+            const float2 a = plane_sum2(x + (size_t)t * row_stride, splits, plane);
+            v[0] = a.x;
+            v[1] = a.y;
+        } else {
+            v[0] = plane_sum(x + (size_t)t * row_stride, splits, plane);
+        }
     };
     // a request's tokens of the tile at a time: the window before the first of them, then eight tokens in flight
     for (int t = tb; t < te;) {
@@ -175,24 +217,59 @@ state_space_operands_kernel(const float *src, int splits, int row_stride, const 
         for (int i = 0; i < W; i++) {
             // place i holds the input W - i tokens back; the shift below brings it to place i - 1
             const int back = W - i, tp = t - back;
-            if (back <= K) win[i] = tp >= t0 ? input(tp) : old[(size_t)(tp - t0 + K) * CC];
+            if (back <= K) {
+                float v[V];
+                if (tp >= t0) {
+                    input(tp, v);
+                } else {
+#pragma unroll
+                    for (int c = 0; c < V; c++) v[c] = old[(size_t)(tp - t0 + K) * CC + c];
+                }
+#pragma unroll
+                for (int c = 0; c < V; c++) win[c][i] = v[c];
+            }
         }
         for (; t < t1; t += 8) {
-            float xin[8];
+            float xin[8][V];
+            if (splits == 1) {                           // (all eight reads in flight)
 #pragma unroll
-            for (int j = 0; j < 8; j++) xin[j] = t + j < t1 ? input(t + j) : 0.f;
+                for (int j = 0; j < 8; j++) {
+                    if (t + j < t1) {
+                        const float *p = x + (size_t)(t + j) * row_stride;
+                        if constexpr (V == 2) { const float2 a = *(const float2 *)p; xin[j][0] = a.x; xin[j][1] = a.y; }
+                        else xin[j][0] = p[0];
+                    }
+                }
+            } else {
+#pragma unroll 1
+                for (int j = 0; j < 8 && t + j < t1; j++) {
+                    float v[V];
+                    input(t + j, v);
+#pragma unroll
+                    for (int jj = 0; jj < 8; jj++)
+                        if (jj == j)
+#pragma unroll
+                            for (int c = 0; c < V; c++) xin[jj][c] = v[c];
+                }
+            }
 #pragma unroll
             for (int j = 0; j < 8; j++) {
                 if (t + j < t1) {
+                    float y[V];
 #pragma unroll
-                    for (int i = 0; i + 1 < W; i++) win[i] = win[i + 1];
-                    win[W - 1] = xin[j];
-                    float acc = b;
+                    for (int c = 0; c < V; c++) {
 #pragma unroll
-                    for (int i = 0; i < W; i++) acc = fmaf(wv[i], win[i], acc);
+                        for (int i = 0; i + 1 < W; i++) win[c][i] = win[c][i + 1];
+                        win[c][W - 1] = xin[j][c];
+                        float acc = b[c];
+#pragma unroll
+                        for (int i = 0; i < W; i++) acc = fmaf(wv[c][i], win[c][i], acc);
+                        y[c] = silu_for<TO>(acc);
+                    }
                     TO *o = dst + (size_t)(t + j) * dst_stride;
-                    o[0] = from_f32<TO>(acc / (1.0f + expf(-acc)));
-                    for (int i = 1; i <= pad; i++) o[i] = from_f32<TO>(0.f);
+                    if constexpr (V == 2) store2(o, y[0], y[1]);
+                    else o[0] = from_f32<TO>(y[0]);
+                    for (int i = V; i < V + pad; i++) o[i] = from_f32<TO>(0.f);
                 }
             }
         }
@@ -201,7 +278,10 @@ state_space_operands_kernel(const float *src, int splits, int row_stride, const 
 #pragma unroll
             for (int i = 0; i < W; i++) {
                 const int back = W - 1 - i;                  // 0: the token itself
-                if (back < K) old[(size_t)(K - 1 - back) * CC] = win[i];
+                if (back < K) {
+#pragma unroll
+                    for (int c = 0; c < V; c++) old[(size_t)(K - 1 - back) * CC + c] = win[c][i];
+                }
             }
         }
     }
@@ -412,7 +492,7 @@ decay_chunk_state_kernel(const __nv_bfloat16 *k, const __nv_bfloat16 *u, const f
 #pragma unroll
         for (int i = 0; i < 4; i++) {
             const int t = ta + (i & 1) + (i >> 1) * 8;
-            wgt[i] = expf(lend - Ls[t]) * cs[t];
+            wgt[i] = __expf(lend - Ls[t]) * cs[t];
         }
 #pragma unroll
         for (int i = 0; i < 4; i++) {                                        // registers: (rows, tokens ta..), (rows + 8, ..), (rows, ta + 8..), ..
@@ -486,30 +566,34 @@ decay_chunk_pass_kernel(const float *__restrict__ dS, const float *__restrict__ 
     *st = S;
 }
 
-// The outputs of a chunk.  Block: chunk x head x 64 value channels; a warp takes 16 tokens.
+// The outputs of a chunk.  A block takes one chunk and one query/key head, whose queries it holds in registers (NK tiles of
+// 16 key channels) and whose scores q . k it computes once; then it walks its share of the (head, 64 value channels) items
+// that read this query/key head, the next item's state and values on their way while it works on one.  A warp takes 16
+// tokens.
+template <int NK>
 __global__ void __launch_bounds__(128)
 decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __nv_bfloat16 *u, const float *la, int la_stride,
                        const float *step, const float *skip, const __nv_bfloat16 *start, const int32_t *chunk_t0, const int32_t *chunk_n,
-                       float *o, int H, int Hq, int dp, int dv, int dvp)
+                       float *o, int H, int Hq, int dp, int dv, int dvp, int v_tiles, int per_block)
 {
     pdl_wait();
     extern __shared__ __align__(16) uint8_t ds_smem[];
     const int P = dp + 8;
-    __nv_bfloat16 *qs = (__nv_bfloat16 *)ds_smem;                            // [CH][P]
-    __nv_bfloat16 *ks = qs + DS_CH * P;                                      // [CH][P]
-    __nv_bfloat16 *sh = ks + DS_CH * P, *sl = sh + DS_DVT * P;               // [DVT][P] each
-    __nv_bfloat16 *us = sl + DS_DVT * P;                                     // [CH][DVT + 8]
-    __shared__ float Ls[DS_CH], cs[DS_CH];
-    const int chunk = blockIdx.x, h = blockIdx.y, hq = h / (H / Hq), v0 = blockIdx.z * DS_DVT;
-    const int vt = min(DS_DVT, dvp - v0);
+    const int stage_elems = 2 * DS_DVT * P + DS_CH * (DS_DVT + 8);
+    __nv_bfloat16 *ks = (__nv_bfloat16 *)ds_smem;                            // [CH][P]
+    __nv_bfloat16 *stages = ks + DS_CH * P;                                  // per stage: sh, sl [DVT][P], us [CH][DVT + 8]
+    __shared__ float Ls[2][DS_CH], cs[2][DS_CH];
+    const int chunk = blockIdx.x, rep = H / Hq, items = rep * v_tiles, shares = (items + per_block - 1) / per_block;
+    const int hq = blockIdx.y / shares, i0 = (blockIdx.y % shares) * per_block, i1 = min(items, i0 + per_block);
     const int t0 = chunk_t0[chunk], n = chunk_n[chunk];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    stage_rows(qs, q + ((size_t)t0 * Hq + hq) * dp, (size_t)Hq * dp, n, DS_CH, dp);
-    stage_rows(ks, k + ((size_t)t0 * Hq + hq) * dp, (size_t)Hq * dp, n, DS_CH, dp);
-    const __nv_bfloat16 *sp = start + ((size_t)chunk * H + h) * 2 * dvp * dp + (size_t)v0 * dp;
-    stage_rows(sh, sp, dp, vt, vt, dp);
-    stage_rows(sl, sp + (size_t)dvp * dp, dp, vt, vt, dp);
-    {
+
+    auto issue = [&](int item, int stage) {
+        const int h = hq * rep + item / v_tiles, v0 = item % v_tiles * DS_DVT, vt = min(DS_DVT, dvp - v0);
+        __nv_bfloat16 *sh = stages + stage * stage_elems, *sl = sh + DS_DVT * P, *us = sl + DS_DVT * P;
+        const __nv_bfloat16 *sp = start + ((size_t)chunk * H + h) * 2 * dvp * dp + (size_t)v0 * dp;
+        stage_rows(sh, sp, dp, vt, vt, dp);
+        stage_rows(sl, sp + (size_t)dvp * dp, dp, vt, vt, dp);
         const int per = vt / 8;
         for (int idx = threadIdx.x; idx < DS_CH * per; idx += 128) {
             const int r = idx / per, c = (idx - r * per) * 8;
@@ -517,97 +601,146 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
             if (r < n) cp16(dst, u + ((size_t)(t0 + r) * H + h) * dvp + v0 + c);
             else *(uint4 *)dst = make_uint4(0, 0, 0, 0);
         }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        chunk_decays(la, la_stride, step, H, h, t0, n, Ls[stage], cs[stage]);        // (the first warp, which has the least to do)
+    };
+    stage_rows(ks, k + ((size_t)t0 * Hq + hq) * dp, (size_t)Hq * dp, n, DS_CH, dp);
+    issue(i0, 0);
+    const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;                    // this thread's two tokens
+    const int nkk = dp / 16;
+    uint32_t qf[NK][4];
+    {
+        const __nv_bfloat16 *q0 = q + ((size_t)(t0 + min(r0, n - 1)) * Hq + hq) * dp + (lane & 3) * 2;
+        const __nv_bfloat16 *q1 = q + ((size_t)(t0 + min(r1, n - 1)) * Hq + hq) * dp + (lane & 3) * 2;
+#pragma unroll
+        for (int kk = 0; kk < NK; kk++) {
+            const bool in = kk < nkk;
+            qf[kk][0] = in ? *(const uint32_t *)(q0 + kk * 16) : 0u;
+            qf[kk][1] = in ? *(const uint32_t *)(q1 + kk * 16) : 0u;
+            qf[kk][2] = in ? *(const uint32_t *)(q0 + kk * 16 + 8) : 0u;
+            qf[kk][3] = in ? *(const uint32_t *)(q1 + kk * 16 + 8) : 0u;
+        }
     }
-    chunk_decays(la, la_stride, step, H, h, t0, n, Ls, cs);
-    cp_wait_all();
-    __syncthreads();
-    if (warp * 16 >= n) return;
-    const float dsk = skip ? skip[h] : 0.f;
-    float acc[8][4];
+    const uint32_t nk = (((lane & 7) + (lane >> 4) * 8) * P + ((lane >> 3) & 1) * 8) * 2;      // [n][k] operands
+    const uint32_t ka = smem_addr(ks) + nk;
+    const bool works = warp * 16 < n;
+    float s[8][4];
 #pragma unroll
     for (int i = 0; i < 8; i++)
 #pragma unroll
-        for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
-    const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;                    // this thread's two tokens
-    const uint32_t qa = smem_addr(qs) + ((warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * P + (lane >> 4) * 8) * 2;
-    const uint32_t nk = (((lane & 7) + (lane >> 4) * 8) * P + ((lane >> 3) & 1) * 8) * 2;      // [n][k] operands
-    const uint32_t ha = smem_addr(sh) + nk, lo_a = smem_addr(sl) + nk, ka = smem_addr(ks) + nk;
-    const uint32_t ua = smem_addr(us) + (((lane & 7) + ((lane >> 3) & 1) * 8) * (DS_DVT + 8) + (lane >> 4) * 8) * 2;
-    const int nkk = dp / 16;
-    // what the state at the chunk's start gives
-    for (int kk = 0; kk < nkk; kk++) {
-        uint32_t a[4];
-        ldsm4(a, qa + kk * 32);
+        for (int j = 0; j < 4; j++) s[i][j] = 0.f;
+    for (int item = i0; item < i1; item++) {
+        const int stage = (item - i0) & 1;
+        if (item + 1 < i1) {
+            issue(item + 1, stage ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        if (works) {
+            if (item == i0) {
 #pragma unroll
-        for (int nt = 0; nt < 4; nt++) {
-            if (nt * 16 < vt) {
-                uint32_t b[4];
-                ldsm4(b, ha + nt * 16 * P * 2 + kk * 32);
-                mma16816(acc[2 * nt], a, b[0], b[1]);
-                mma16816(acc[2 * nt + 1], a, b[2], b[3]);
-                ldsm4(b, lo_a + nt * 16 * P * 2 + kk * 32);
-                mma16816(acc[2 * nt], a, b[0], b[1]);
-                mma16816(acc[2 * nt + 1], a, b[2], b[3]);
+                for (int kt = 0; kt < 4; kt++) {
+                    if (kt <= warp) {
+#pragma unroll
+                        for (int kk = 0; kk < NK; kk++) {
+                            if (kk < nkk) {
+                                uint32_t b[4];
+                                ldsm4(b, ka + kt * 16 * P * 2 + kk * 32);
+                                mma16816(s[2 * kt], qf[kk], b[0], b[1]);
+                                mma16816(s[2 * kt + 1], qf[kk], b[2], b[3]);
+                            }
+                        }
+                    }
+                }
+            }
+            const int h = hq * rep + item / v_tiles, v0 = item % v_tiles * DS_DVT, vt = min(DS_DVT, dvp - v0);
+            const __nv_bfloat16 *sh = stages + stage * stage_elems, *sl = sh + DS_DVT * P, *us = sl + DS_DVT * P;
+            const uint32_t ha = smem_addr(sh) + nk, lo_a = smem_addr(sl) + nk;
+            const uint32_t ua = smem_addr(us) + (((lane & 7) + ((lane >> 3) & 1) * 8) * (DS_DVT + 8) + (lane >> 4) * 8) * 2;
+            const float dsk = skip ? skip[h] : 0.f;
+            float acc[8][4];
+#pragma unroll
+            for (int i = 0; i < 8; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
+            // what the state at the chunk's start gives
+#pragma unroll
+            for (int kk = 0; kk < NK; kk++) {
+                if (kk < nkk) {
+#pragma unroll
+                    for (int nt = 0; nt < 4; nt++) {
+                        if (nt * 16 < vt) {
+                            uint32_t b[4], c[4];
+                            ldsm4(b, ha + nt * 16 * P * 2 + kk * 32);
+                            ldsm4(c, lo_a + nt * 16 * P * 2 + kk * 32);
+                            mma16816(acc[2 * nt], qf[kk], b[0], b[1]);
+                            mma16816(acc[2 * nt + 1], qf[kk], b[2], b[3]);
+                            mma16816(acc[2 * nt], qf[kk], c[0], c[1]);
+                            mma16816(acc[2 * nt + 1], qf[kk], c[2], c[3]);
+                        }
+                    }
+                }
+            }
+            const float L0 = Ls[stage][r0], L1 = Ls[stage][r1];
+            {
+                const float e0 = __expf(L0), e1 = __expf(L1);
+#pragma unroll
+                for (int i = 0; i < 8; i++) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
+            }
+            // what the chunk's own tokens give
+#pragma unroll
+            for (int kt = 0; kt < 4; kt++) {
+                if (kt <= warp) {
+                    uint32_t hi[4], lo[4];
+#pragma unroll
+                    for (int half = 0; half < 2; half++) {
+                        const int key = kt * 16 + half * 8 + (lane & 3) * 2;
+                        const float2 Lk = *(const float2 *)&Ls[stage][key], ck = *(const float2 *)&cs[stage][key];
+                        float w[4];
+#pragma unroll
+                        for (int i = 0; i < 4; i++) {
+                            const int ky = key + (i & 1), r = i < 2 ? r0 : r1;
+                            const float L = (i < 2 ? L0 : L1) - (i & 1 ? Lk.y : Lk.x);
+                            float v = ky <= r ? s[2 * kt + half][i] * __expf(fminf(L, 0.f)) * (i & 1 ? ck.y : ck.x) : 0.f;
+                            if (ky == r) v += dsk;
+                            w[i] = v;
+                        }
+                        split2(w[0], w[1], hi[2 * half], lo[2 * half]);
+                        split2(w[2], w[3], hi[2 * half + 1], lo[2 * half + 1]);
+                    }
+#pragma unroll
+                    for (int nt = 0; nt < 4; nt++) {
+                        if (nt * 16 < vt) {
+                            uint32_t b[4];
+                            ldsm4_t(b, ua + (kt * 16 * (DS_DVT + 8) + nt * 16) * 2);
+                            mma16816(acc[2 * nt], hi, b[0], b[1]);
+                            mma16816(acc[2 * nt + 1], hi, b[2], b[3]);
+                            mma16816(acc[2 * nt], lo, b[0], b[1]);
+                            mma16816(acc[2 * nt + 1], lo, b[2], b[3]);
+                        }
+                    }
+                }
+            }
+            const bool even = (dv & 1) == 0;
+#pragma unroll
+            for (int nt = 0; nt < 8; nt++) {
+                const int c = v0 + nt * 8 + (lane & 3) * 2;
+                if (nt * 8 < vt && c < dv) {
+#pragma unroll
+                    for (int half = 0; half < 2; half++) {
+                        const int r = half ? r1 : r0;
+                        if (r < n) {
+                            float *p = o + ((size_t)(t0 + r) * H + h) * dv + c;
+                            if (even) *(float2 *)p = make_float2(acc[nt][2 * half], acc[nt][2 * half + 1]);
+                            else { p[0] = acc[nt][2 * half]; if (c + 1 < dv) p[1] = acc[nt][2 * half + 1]; }
+                        }
+                    }
+                }
             }
         }
-    }
-    const float L0 = Ls[r0], L1 = Ls[r1];
-    {
-        const float e0 = expf(L0), e1 = expf(L1);
-#pragma unroll
-        for (int i = 0; i < 8; i++) { acc[i][0] *= e0; acc[i][1] *= e0; acc[i][2] *= e1; acc[i][3] *= e1; }
-    }
-    // what the chunk's own tokens give
-    for (int kt = 0; kt <= warp; kt++) {
-        float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-        for (int kk = 0; kk < nkk; kk++) {
-            uint32_t a[4], b[4];
-            ldsm4(a, qa + kk * 32);
-            ldsm4(b, ka + kt * 16 * P * 2 + kk * 32);
-            mma16816(s[0], a, b[0], b[1]);
-            mma16816(s[1], a, b[2], b[3]);
-        }
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int key = kt * 16 + half * 8 + (lane & 3) * 2;
-            float w[4];
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                const int ky = key + (i & 1), r = i < 2 ? r0 : r1;
-                const float L = i < 2 ? L0 : L1;
-                float v = ky <= r ? s[half][i] * expf(fminf(L - Ls[ky], 0.f)) * cs[ky] : 0.f;
-                if (ky == r) v += dsk;
-                w[i] = v;
-            }
-            split2(w[0], w[1], hi[2 * half], lo[2 * half]);
-            split2(w[2], w[3], hi[2 * half + 1], lo[2 * half + 1]);
-        }
-#pragma unroll
-        for (int nt = 0; nt < 4; nt++) {
-            if (nt * 16 < vt) {
-                uint32_t b[4];
-                ldsm4_t(b, ua + (kt * 16 * (DS_DVT + 8) + nt * 16) * 2);
-                mma16816(acc[2 * nt], hi, b[0], b[1]);
-                mma16816(acc[2 * nt], lo, b[0], b[1]);
-                mma16816(acc[2 * nt + 1], hi, b[2], b[3]);
-                mma16816(acc[2 * nt + 1], lo, b[2], b[3]);
-            }
-        }
-    }
-    const bool even = (dv & 1) == 0;
-#pragma unroll
-    for (int nt = 0; nt < 8; nt++) {
-        const int c = v0 + nt * 8 + (lane & 3) * 2;
-        if (nt * 8 >= vt || c >= dv) continue;
-#pragma unroll
-        for (int half = 0; half < 2; half++) {
-            const int r = half ? r1 : r0;
-            if (r >= n) continue;
-            float *p = o + ((size_t)(t0 + r) * H + h) * dv + c;
-            if (even) *(float2 *)p = make_float2(acc[nt][2 * half], acc[nt][2 * half + 1]);
-            else { p[0] = acc[nt][2 * half]; if (c + 1 < dv) p[1] = acc[nt][2 * half + 1]; }
-        }
+        __syncthreads();                                                     // the stage is free for the item after the next
     }
 }
 
@@ -615,51 +748,43 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
 // A row of o [T, C] in parts of n values, each divided by its own root mean square; the gate silu(g) multiplies before the
 // norm (gate_first) or after it; times a weight [C] where there is one.  g is the sum of `splits` planes [T, g_stride] read
 // from column g_col0 on.  TH threads per part, at most 16 values a thread, V at a time.
-template <typename TO, int TH, int V>
+template <typename TO, int TH, int V, int N>
 __global__ void __launch_bounds__(TH < 128 ? 128 : TH)
 part_norm_gate_kernel(const float *o, const float *g, int splits, int g_stride, int g_col0, const float *w, float eps, int gate_first,
                       TO *out, size_t out_stride, int T, int C, int n, int parts)
 {
     pdl_entry();
     pdl_sync_small();
-    constexpr int PER_BLOCK = TH < 128 ? 128 / TH : 1, N = 16 / V;
+    constexpr int PER_BLOCK = TH < 128 ? 128 / TH : 1;
     const int lane = threadIdx.x % TH, p = blockIdx.y * PER_BLOCK + threadIdx.x / TH, t = blockIdx.x;
     __shared__ float red[32];
     if (PER_BLOCK > 1 && p >= parts) return;
     const size_t plane = (size_t)T * g_stride;
     const float *op = o + (size_t)t * C + (size_t)p * n, *gp = g + (size_t)t * g_stride + g_col0 + (size_t)p * n;
-    float v[16], gate[16];
+    float v[N * V], gate[N * V];
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < N; j++) {
         const int c = (lane + j * TH) * V;
         if (c < n) {
             if constexpr (V == 4) {
-                const float4 a = *(const float4 *)(op + c);
-                float4 z = *(const float4 *)(gp + c);
-                for (int s = 1; s < splits; s++) {
-                    const float4 y = *(const float4 *)(gp + (size_t)s * plane + c);
-                    z.x += y.x; z.y += y.y; z.z += y.z; z.w += y.w;
-                }
+                const float4 a = *(const float4 *)(op + c), z = plane_sum4(gp + c, splits, plane);
                 v[4 * j] = a.x; v[4 * j + 1] = a.y; v[4 * j + 2] = a.z; v[4 * j + 3] = a.w;
                 gate[4 * j] = z.x; gate[4 * j + 1] = z.y; gate[4 * j + 2] = z.z; gate[4 * j + 3] = z.w;
             } else {
                 v[j] = op[c];
-                float z = gp[c];
-                for (int s = 1; s < splits; s++) z += gp[(size_t)s * plane + c];
-                gate[j] = z;
+                gate[j] = plane_sum(gp + c, splits, plane);
             }
         } else {
 #pragma unroll
             for (int i = 0; i < V; i++) { v[V * j + i] = 0.f; gate[V * j + i] = 0.f; }
         }
+    }
 #pragma unroll
-        for (int i = 0; i < V; i++) {
-            const float z = gate[V * j + i];
-            gate[V * j + i] = z / (1.0f + expf(-z));
-            if (gate_first) v[V * j + i] *= gate[V * j + i];
-            ss = fmaf(v[V * j + i], v[V * j + i], ss);
-        }
+    for (int j = 0; j < N * V; j++) {
+        gate[j] = silu_for<TO>(gate[j]);
+        if (gate_first) v[j] *= gate[j];
+        ss = fmaf(v[j], v[j], ss);
     }
     ss = warp_sum(ss);
     if (TH > 32) {
@@ -681,22 +806,13 @@ part_norm_gate_kernel(const float *o, const float *g, int splits, int g_stride, 
             v[V * j + i] = y;
         }
         if constexpr (V == 4) {
-            if constexpr (sizeof(TO) == 4) {
-                *(float4 *)((float *)(void *)dst + c) = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
-            } else {
-                const __nv_bfloat162 a = __floats2bfloat162_rn(v[4 * j], v[4 * j + 1]), b = __floats2bfloat162_rn(v[4 * j + 2], v[4 * j + 3]);
-                uint2 y;
-                y.x = *(const uint32_t *)&a;
-                y.y = *(const uint32_t *)&b;
-                *(uint2 *)(void *)(dst + c) = y;
-            }
+            store2(dst + c, v[4 * j], v[4 * j + 1]);
+            store2(dst + c + 2, v[4 * j + 2], v[4 * j + 3]);
         } else {
             dst[c] = from_f32<TO>(v[j]);
         }
     }
 }
-
-static bool aligned16(const void *p) { return ((uintptr_t)p & 15) == 0; }
 
 }  // namespace hfb
 
@@ -722,13 +838,16 @@ extern "C" int hfb_rotate_heads(const float *src, int splits, int row_stride, co
         !q || !k || !u || !valid_dt(out_dt))
         return fail(HFB_EINVAL, "rotate_heads: bad arguments (n_rot=%d)", n_rot);
     const dim3 grid(T, (H + 3) / 4);
+    // (dp and dvp are multiples of 16, the outputs' heads therefore aligned)
+    const int pairs = (d & 1) == 0 && (dv & 1) == 0 && (row_stride & 1) == 0 && (n_rot & 3) == 0 && ((uintptr_t)src & 7) == 0 && aligned16(cos_sin) &&
+                      aligned16(q) && aligned16(k) && aligned16(u);
     if (out_dt == HFB_F32)
         g_launch_err = launch_pdl(rotate_heads_kernel<float>, grid, dim3(128), 0, (cudaStream_t)s, src, splits, row_stride, cos_sin, n_rot, n_positions,
-                                  positions, k_scale, (float *)q, (float *)k, (float *)u, T, H, d, dv, dp, dvp, error_word());
+                                  positions, k_scale, (float *)q, (float *)k, (float *)u, T, H, d, dv, dp, dvp, pairs, error_word());
     else
         g_launch_err = launch_pdl(rotate_heads_kernel<__nv_bfloat16>, grid, dim3(128), 0, (cudaStream_t)s, src, splits, row_stride, cos_sin, n_rot,
                                   n_positions, positions, k_scale, (__nv_bfloat16 *)q, (__nv_bfloat16 *)k, (__nv_bfloat16 *)u, T, H, d, dv, dp,
-                                  dvp, error_word());
+                                  dvp, pairs, error_word());
     return check_pdl_launch(g_launch_err, "rotate_heads");
 }
 
@@ -747,17 +866,21 @@ extern "C" int hfb_state_space_operands(const float *src, int splits, int row_st
         return fail(HFB_EINVAL, "state_space_operands: bad arguments (taps=%d)", taps);
     if (taps > DS_MAX_TAPS) return fail(HFB_ENOTSUP, "state_space_operands: %d taps exceed %d", taps, DS_MAX_TAPS);
     const int single = T == S;                           // every request brings one token
-    const int blocks_x = (CC + 127) / 128 + (H + 127) / 128;
+    const bool two = (d & 1) == 0 && (dv & 1) == 0 && (row_stride & 1) == 0 && ((uintptr_t)src & 7) == 0 && aligned16(q) && aligned16(k) && aligned16(u);
+    const int per = two ? 256 : 128;
+    const int blocks_x = (CC + per - 1) / per + (H + 127) / 128;
     int tt = 32;                                         // tokens of a block: fewer where that leaves SMs idle
     while (tt > 1 && (long)blocks_x * ((T + tt - 1) / tt) < 148 * 8) tt >>= 1;
     if ((T + tt - 1) / tt > 65535) tt = (T + 65534) / 65535;
     const dim3 grid(blocks_x, (T + tt - 1) / tt);
-#define HFB_SSO(TAPS, TY) \
-    g_launch_err = launch_pdl(state_space_operands_kernel<TAPS, TY>, grid, dim3(128), 0, (cudaStream_t)s, src, splits, row_stride, w, w_dt, bias, bias_dt, \
+#define HFB_SSO(TAPS, V, TY) \
+    g_launch_err = launch_pdl(state_space_operands_kernel<TAPS, V, TY>, grid, dim3(128), 0, (cudaStream_t)s, src, splits, row_stride, w, w_dt, bias, bias_dt, \
                               taps, dt_bias, dtb_dt, rate, carried, (size_t)slot_stride, token_seq, cu_tokens, seq_slots, n_slots, single, (TY *)q, \
                               (TY *)k, (TY *)u, step, la, T, H, G, d, dv, dp, dvp, tt, error_word())
-    if (out_dt == HFB_F32) { if (taps == 4) HFB_SSO(4, float); else HFB_SSO(0, float); }
-    else { if (taps == 4) HFB_SSO(4, __nv_bfloat16); else HFB_SSO(0, __nv_bfloat16); }
+#define HFB_SSOT(TY) do { if (taps == 4 && two) HFB_SSO(4, 2, TY); else if (taps == 4) HFB_SSO(4, 1, TY); else if (two) HFB_SSO(0, 2, TY); else HFB_SSO(0, 1, TY); } while (0)
+    if (out_dt == HFB_F32) HFB_SSOT(float);
+    else HFB_SSOT(__nv_bfloat16);
+#undef HFB_SSOT
 #undef HFB_SSO
     rc = check_pdl_launch(g_launch_err, "state_space_operands");
     if (rc != HFB_OK || single) return rc;
@@ -831,18 +954,30 @@ extern "C" int hfb_decay_chunks(const void *q, const void *k, const void *u, con
     g_launch_err = launch_pdl(decay_chunk_pass_kernel, dim3((unsigned)((st / 4 + 255) / 256), S), dim3(256), 0, (cudaStream_t)s, dS, l_end, state,
                               (size_t)slot_stride, chunk_first, seq_slots, n_slots, start, H, dp, dvp, error_word());
     if ((rc = check_pdl_launch(g_launch_err, "decay_chunk_pass")) != HFB_OK) return rc;
-    const size_t smem_c = ((size_t)2 * (DS_CH + DS_DVT) * (dp + 8) + (size_t)DS_CH * (DS_DVT + 8)) * 2;
-    static bool opted[64] = {false};
-    const int dev = current_device();
-    if (!opted[dev]) {
-        const int most = (2 * (DS_CH + DS_DVT) * (DS_MAX_CHUNK_D + 8) + DS_CH * (DS_DVT + 8)) * 2;
-        cudaError_t e = cudaFuncSetAttribute(decay_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
-        if (e != cudaSuccess) return fail(HFB_ECUDA, "decay_chunks: %s", cudaGetErrorString(e));
-        opted[dev] = true;
-    }
-    g_launch_err = launch_pdl(decay_chunk_out_kernel, dim3(chunks, H, v_tiles), dim3(128), smem_c, (cudaStream_t)s, (const __nv_bfloat16 *)q,
-                              (const __nv_bfloat16 *)k, (const __nv_bfloat16 *)u, la, la_stride, step, skip, start, chunk_t0, chunk_n, o, H, Hq, dp,
-                              dv, dvp);
+    const size_t smem_c = ((size_t)DS_CH * (dp + 8) + 2 * ((size_t)2 * DS_DVT * (dp + 8) + (size_t)DS_CH * (DS_DVT + 8))) * 2;
+    // a block's share of the items that read one query/key head: as many as leave four blocks for every SM
+    const int items = H / Hq * v_tiles;
+    int per_block = items < 8 ? items : 8;
+    while (per_block > 1 && (long)chunks * Hq * ((items + per_block - 1) / per_block) < 148 * 4) per_block--;
+    const int shares = (items + per_block - 1) / per_block;
+    if ((long)Hq * shares > 65535) return fail(HFB_ENOTSUP, "decay_chunks: %d heads exceed the grid limit", H);
+#define HFB_CHUNK_OUT(NK) do { \
+        static bool opted[64] = {false}; \
+        const int dev = current_device(); \
+        if (!opted[dev]) { \
+            const int most = (DS_CH * (NK * 16 + 8) + 2 * (2 * DS_DVT * (NK * 16 + 8) + DS_CH * (DS_DVT + 8))) * 2; \
+            cudaError_t e = cudaFuncSetAttribute(decay_chunk_out_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, most); \
+            if (e != cudaSuccess) return fail(HFB_ECUDA, "decay_chunks: %s", cudaGetErrorString(e)); \
+            opted[dev] = true; \
+        } \
+        g_launch_err = launch_pdl(decay_chunk_out_kernel<NK>, dim3(chunks, Hq * shares), dim3(128), smem_c, (cudaStream_t)s, (const __nv_bfloat16 *)q, \
+                                  (const __nv_bfloat16 *)k, (const __nv_bfloat16 *)u, la, la_stride, step, skip, start, chunk_t0, chunk_n, o, H, Hq, \
+                                  dp, dv, dvp, v_tiles, per_block); \
+    } while (0)
+    if (dp <= 64) HFB_CHUNK_OUT(4);
+    else if (dp <= 128) HFB_CHUNK_OUT(8);
+    else HFB_CHUNK_OUT(16);
+#undef HFB_CHUNK_OUT
     return check_pdl_launch(g_launch_err, "decay_chunk_out");
 }
 
@@ -857,12 +992,20 @@ extern "C" int hfb_part_norm_gate(const float *o, const float *g, int splits, in
     if (parts > 65535) return fail(HFB_ENOTSUP, "part_norm_gate: %d parts exceed the grid limit", parts);
     const bool vec = (n & 3) == 0 && (g_stride & 3) == 0 && (g_col0 & 3) == 0 && aligned16(o) && aligned16(g) && (out_stride & 3) == 0 &&
                      ((uintptr_t)out & (4 * esz - 1)) == 0;
-#define HFB_PNG(TY, TH, V) \
-    g_launch_err = launch_pdl(part_norm_gate_kernel<TY, TH, V>, dim3(T, TH < 128 ? (parts + 128 / TH - 1) / (128 / TH) : parts), dim3(TH < 128 ? 128 : TH), 0, \
-                              (cudaStream_t)s, o, g, splits, g_stride, g_col0, w, eps, gate_first, (TY *)out, (size_t)out_stride, T, C, n, parts)
-#define HFB_PNGT(TY, V) do { if (n <= 512) HFB_PNG(TY, 32, V); else if (n <= 4096) HFB_PNG(TY, 256, V); else HFB_PNG(TY, 1024, V); } while (0)
-    if (out_dt == HFB_F32) { if (vec) HFB_PNGT(float, 4); else HFB_PNGT(float, 1); }
-    else { if (vec) HFB_PNGT(__nv_bfloat16, 4); else HFB_PNGT(__nv_bfloat16, 1); }
+#define HFB_PNG(TY, TH, V, N) \
+    g_launch_err = launch_pdl(part_norm_gate_kernel<TY, TH, V, N>, dim3(T, TH < 128 ? (parts + 128 / TH - 1) / (128 / TH) : parts), dim3(TH < 128 ? 128 : TH), \
+                              0, (cudaStream_t)s, o, g, splits, g_stride, g_col0, w, eps, gate_first, (TY *)out, (size_t)out_stride, T, C, n, parts)
+    // a warp for parts of up to 128, 256 or 512 values, else a block
+#define HFB_PNGT(TY) do { \
+        if (vec) { \
+            if (n <= 128) HFB_PNG(TY, 32, 4, 1); else if (n <= 256) HFB_PNG(TY, 32, 4, 2); else if (n <= 512) HFB_PNG(TY, 32, 4, 4); \
+            else if (n <= 2048) HFB_PNG(TY, 256, 4, 2); else if (n <= 4096) HFB_PNG(TY, 256, 4, 4); else HFB_PNG(TY, 1024, 4, 4); \
+        } else { \
+            if (n <= 512) HFB_PNG(TY, 32, 1, 16); else if (n <= 4096) HFB_PNG(TY, 256, 1, 16); else HFB_PNG(TY, 1024, 1, 16); \
+        } \
+    } while (0)
+    if (out_dt == HFB_F32) HFB_PNGT(float);
+    else HFB_PNGT(__nv_bfloat16);
 #undef HFB_PNGT
 #undef HFB_PNG
     return check_pdl_launch(g_launch_err, "part_norm_gate");

@@ -196,9 +196,19 @@ __device__ __forceinline__ void epilogue_chunk(const GemmParams &p, const uint32
 #pragma unroll
             for (int i = 0; i < 16; i++) f[i] = __uint_as_float(v[i]);
             if (p.bias) {
+                if (p.bias_dt == HFB_BF16 && y0 + 16 <= p.N) {        // (the bias is 16-byte aligned, y0 a multiple of 16)
+                    const uint4 *bp = (const uint4 *)((const __nv_bfloat16 *)p.bias + y0);
+                    const uint4 b0 = bp[0], b1 = bp[1];
+                    const __nv_bfloat162 *h0 = (const __nv_bfloat162 *)&b0, *h1 = (const __nv_bfloat162 *)&b1;
 #pragma unroll
-                for (int i = 0; i < 16; i++)
-                    if (y0 + i < p.N) f[i] += load_any(p.bias, p.bias_dt, y0 + i);
+                    for (int i = 0; i < 4; i++) {
+                        const float2 x = __bfloat1622float2(h0[i]), y = __bfloat1622float2(h1[i]);
+                        f[2 * i] += x.x; f[2 * i + 1] += x.y; f[8 + 2 * i] += y.x; f[8 + 2 * i + 1] += y.y;
+                    }
+                } else {
+                    for (int i = 0; i < 16; i++)
+                        if (y0 + i < p.N) f[i] += load_any(p.bias, p.bias_dt, y0 + i);
+                }
             }
             if (p.act == HFB_ACT_CLAMPED_GLU) {
 #pragma unroll
@@ -1120,7 +1130,7 @@ extern "C" int hfb_linear_tc_glu(const void *a, const void *w, const void *bias,
                                  int N, int K, int act, float limit, float alpha, float offset, hfb_stream s)
 {
     if (M <= 0 || N <= 0) return HFB_OK;
-    int rc = check_tc_args("linear_tc_glu", a, w, out, M, N, K);
+    int rc = check_tc_args("linear_tc_glu", a, w, out, M, N, K, bias);
     if (rc != HFB_OK) return rc;
     if ((N & 1) || !valid_dt(out_dt) || act < 0 || (act >= HFB_ACT_NONE && act != HFB_ACT_CLAMPED_GLU) || (bias && !valid_dt(bias_dt)) ||
         (ldo && ldo < N / 2))

@@ -135,23 +135,6 @@ rope_norm_kv_kernel(const float *src, int splits, const void *bias, int bias_dt,
 // `splits` planes.  q = row / sqrt(mean(row^2) + eps) * q_w over the QD queries, keys likewise with k_w; queries to q_out
 // [T, QD], keys and values to the token's cache slot (KD = VD = 0: the layer reads another layer's cache), gates as
 // sigmoid(row) to gate_out [T, n_gate] float32.  One block per token.
-__device__ __forceinline__ float4 sum_planes4(const float *p, int splits, size_t plane)
-{
-    float4 a = *(const float4 *)p;
-    for (int s = 1; s < splits; s++) {
-        const float4 b = *(const float4 *)(p + (size_t)s * plane);
-        a.x += b.x; a.y += b.y; a.z += b.z; a.w += b.w;
-    }
-    return a;
-}
-
-__device__ __forceinline__ float sum_planes(const float *p, int splits, size_t plane)
-{
-    float a = *p;
-    for (int s = 1; s < splits; s++) a += p[(size_t)s * plane];
-    return a;
-}
-
 template <typename TO>
 __global__ void __launch_bounds__(256)
 row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_w, const float *k_w, float eps, const int32_t *slots,
@@ -170,24 +153,24 @@ row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_
     float sq = 0.f, sk = 0.f;
     if (vec) {
         for (int c = threadIdx.x * 4; c < n; c += 1024) {
-            const float4 v = sum_planes4(row + c, splits, plane);
+            const float4 v = plane_sum4(row + c, splits, plane);
             *(float4 *)(rn_row + c) = v;
             const float ss = (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
             if (c < QD) sq += ss; else sk += ss;
         }
         if (slot >= 0)
-            for (int c = threadIdx.x * 4; c < VD; c += 1024) store4(v_cache + (size_t)slot * VD + c, sum_planes4(row + n + c, splits, plane));
+            for (int c = threadIdx.x * 4; c < VD; c += 1024) store4(v_cache + (size_t)slot * VD + c, plane_sum4(row + n + c, splits, plane));
     } else {
         for (int c = threadIdx.x; c < n; c += 256) {
-            const float v = sum_planes(row + c, splits, plane);
+            const float v = plane_sum(row + c, splits, plane);
             rn_row[c] = v;
             if (c < QD) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
         }
         if (slot >= 0)
-            for (int c = threadIdx.x; c < VD; c += 256) v_cache[(size_t)slot * VD + c] = from_f32<TO>(sum_planes(row + n + c, splits, plane));
+            for (int c = threadIdx.x; c < VD; c += 256) v_cache[(size_t)slot * VD + c] = from_f32<TO>(plane_sum(row + n + c, splits, plane));
     }
     for (int c = threadIdx.x; c < n_gate; c += 256)
-        gate_out[(size_t)t * n_gate + c] = 1.0f / (1.0f + expf(-sum_planes(row + n + VD + c, splits, plane)));
+        gate_out[(size_t)t * n_gate + c] = 1.0f / (1.0f + expf(-plane_sum(row + n + VD + c, splits, plane)));
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;

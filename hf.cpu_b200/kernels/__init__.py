@@ -200,6 +200,18 @@ def set_launch_overlap(on: bool) -> None:
         fn(bool(on))
 
 
+def run_beside(first, second) -> None:
+    """Runs two pieces of work that do not depend on one another.  While a step is being captured as a graph they become two
+    branches of it, so that one's kernels may run beside the other's; else one after the other.  They must not share scratch
+    (``second`` makes no split product: the partial sums have one workspace)."""
+    b = backend()
+    if hasattr(b, "run_beside"):
+        b.run_beside(first, second)
+    else:
+        first()
+        second()
+
+
 def paged_attention(q, k_cache, v_cache, meta, ctx, H, G, d, window, scale, out, tiles=None, dv=None, values_in_keys=False,
                     sinks=None, zero_sink=False, slopes=None, head_scales=None, softcap: float = 0.0) -> None:
     """``window``: a :func:`mask_code`.  ``tiles``: the device arrays of :func:`attention_step_arrays` for this step

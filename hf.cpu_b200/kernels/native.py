@@ -72,6 +72,8 @@ class NativeBackend:
         self.merge_in_kernel = True
         self.rope_in_epilogue = os.environ.get("HFB_ROPE_EPILOGUE", "1") != "0"     # prompts: q|k|v product rotates and writes the cache
         self._counters = None
+        self.branches = os.environ.get("HFB_BRANCHES", "1") != "0"        # independent work of a captured step as branches of the graph
+        self._side = None
         self.lib.hfb_linear_tc_partials_workspace.restype = ctypes.c_size_t
         self.lib.hfb_argmax2_scratch.restype = ctypes.c_size_t
         self.lib.hfb_decay_chunks_scratch.restype = ctypes.c_size_t
@@ -161,6 +163,20 @@ class NativeBackend:
                                                _p(positions), _p(slots), _p(q_out), _p(k_cache), _p(v_cache),
                                                c_int64(cache_slots), c_int(T), c_int(H), c_int(G), c_int(d),
                                                self._stream()), "rope_kv_write")
+
+    def run_beside(self, first, second):
+        if not self.branches or not torch.cuda.is_current_stream_capturing():
+            first()
+            second()
+            return
+        here = torch.cuda.current_stream()
+        if self._side is None:
+            self._side = torch.cuda.Stream()
+        self._side.wait_stream(here)
+        with torch.cuda.stream(self._side):
+            second()
+        first()
+        here.wait_stream(self._side)
 
     def set_launch_overlap(self, on):
         self.lib.hfb_set_launch_overlap(c_int(1 if on else 0))

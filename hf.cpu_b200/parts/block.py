@@ -139,8 +139,11 @@ class ParallelResidual(Block):
     """``x += mixer(h) + ffn(h)``, ``h = norm1(x)``: both sublayers read the same normed input, there is no second norm, and a
     layer may have no feed-forward.  Where both sublayers offer the operand of their last product, the two operands lie
     side by side in one buffer and ONE product over the joined inner dimension ([W_o | W_down] [att; hidden]) ends the
-    layer: one pass over the stream, one sum in float32, the following norm in its tail."""
+    layer: one pass over the stream, one sum in float32, the following norm in its tail.  In a captured step the two
+    operands are made on two branches of the graph (the mixer's chain of short kernels beside the feed-forward's product);
+    its launches therefore do not overlap with the kernel in front of them."""
     graph_safe = True
+    launch_overlap_safe = False
 
     def __init__(self, **_):
         self.w_out = self.b_out = None
@@ -167,8 +170,7 @@ class ParallelResidual(Block):
         if self.widths is not None:
             m, f = self.widths
             both = ctx.buf("block_operand", (x.shape[0], m + f), ctx.run_dtype)
-            mixer.operand(ctx, xn, cache, state, write_cache, both[:, :m])
-            ffn.operand(ctx, xn, both[:, m:])
+            kernels.run_beside(lambda: mixer.operand(ctx, xn, cache, state, write_cache, both[:, :m]), lambda: ffn.operand(ctx, xn, both[:, m:]))
             args = next_norm.fused_args() if next_norm is not None else None
             with kernels.phase("down"):
                 if args is None:
