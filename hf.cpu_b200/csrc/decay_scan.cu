@@ -30,7 +30,6 @@ int *error_word();
 
 constexpr int DS_CH = 64;             // tokens of a chunk
 constexpr int DS_DVT = 64;            // value channels of a block
-constexpr int DS_DT = 128;            // key channels of a block of the state kernel
 constexpr int DS_MAX_CHUNK_D = 256;   // largest padded key head of the chunk form
 constexpr int DS_MAX_D = 512;         // ... and of the walk
 constexpr int DS_MAX_TAPS = 16;
@@ -405,27 +404,38 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t &hi, uint32_t 
     lo = *(const uint32_t *)&l;
 }
 
-// Rows [n rows of `cols` values, row_stride apart] to shared memory rows of cols + 8 values, rows beyond n as zeros.
+// `rows` x COLS values of shared memory (rows COLS + 8 values apart) from n rows of `cols` values, row_stride apart, zeros
+// beyond them.
+template <int COLS>
 __device__ __forceinline__ void stage_rows(__nv_bfloat16 *dst, const __nv_bfloat16 *src, size_t row_stride, int n, int rows, int cols)
 {
-    const int per = cols / 8;
-    for (int idx = threadIdx.x; idx < rows * per; idx += blockDim.x) {
-        const int r = idx / per, c = (idx - r * per) * 8;
-        if (r < n) cp16(dst + r * (cols + 8) + c, src + (size_t)r * row_stride + c);
-        else *(uint4 *)(dst + r * (cols + 8) + c) = make_uint4(0, 0, 0, 0);
+    constexpr int PER = COLS / 8;
+#pragma unroll 4
+    for (int idx = threadIdx.x; idx < rows * PER; idx += 128) {
+        const int r = idx / PER, c = idx % PER * 8;
+        __nv_bfloat16 *to = dst + r * (COLS + 8) + c;
+        if (r < n && c < cols) cp16(to, src + (size_t)r * row_stride + c);
+        else *(uint4 *)to = make_uint4(0, 0, 0, 0);
     }
 }
 
-// L[i] = la summed over the chunk's tokens 0 .. i (first warp; tokens beyond n repeat the last sum), c[i] = step sizes (1
-// where there are none, 0 beyond n).  The caller synchronises.
-__device__ __forceinline__ void chunk_decays(const float *la, int la_stride, const float *step, int H, int h, int t0, int n, float *Ls, float *cs)
-{
-    if (threadIdx.x < 32) {
+// Decays of a chunk, by the first warp: two tokens' la and step size a lane (1 where there are no step sizes, 0 beyond n),
+// then L[i] = la summed over the tokens 0 .. i (tokens beyond n repeat the last sum) and c[i] = step sizes.
+struct ChunkDecays {
+    float a, b, ca, cb;
+    __device__ __forceinline__ void fetch(const float *la, int la_stride, const float *step, int H, int h, int t0, int n)
+    {
         const int i = threadIdx.x * 2;
-        float a = i < n ? la[(size_t)(t0 + i) * la_stride + h] : 0.f;
-        float b = i + 1 < n ? la[(size_t)(t0 + i + 1) * la_stride + h] : 0.f;
-        b += a;
-        float run = b;
+        a = i < n ? la[(size_t)(t0 + i) * la_stride + h] : 0.f;
+        b = i + 1 < n ? la[(size_t)(t0 + i + 1) * la_stride + h] : 0.f;
+        ca = i < n ? (step ? step[(size_t)(t0 + i) * H + h] : 1.0f) : 0.f;
+        cb = i + 1 < n ? (step ? step[(size_t)(t0 + i + 1) * H + h] : 1.0f) : 0.f;
+    }
+    __device__ __forceinline__ void finish(float *Ls, float *cs) const
+    {
+        const int i = threadIdx.x * 2;
+        const float both = a + b;
+        float run = both;
 #pragma unroll
         for (int m = 1; m < 32; m <<= 1) {
             const float v = __shfl_up_sync(0xffffffffu, run, m);
@@ -434,65 +444,57 @@ __device__ __forceinline__ void chunk_decays(const float *la, int la_stride, con
         const float before = __shfl_up_sync(0xffffffffu, run, 1);
         const float base = threadIdx.x ? before : 0.f;
         Ls[i] = base + a;
-        Ls[i + 1] = base + b;
-        cs[i] = i < n ? (step ? step[(size_t)(t0 + i) * H + h] : 1.0f) : 0.f;
-        cs[i + 1] = i + 1 < n ? (step ? step[(size_t)(t0 + i + 1) * H + h] : 1.0f) : 0.f;
+        Ls[i + 1] = base + both;
+        cs[i] = ca;
+        cs[i + 1] = cb;
     }
-}
+};
 
 // What a chunk adds to the state: dS[chunk][h][dvp][dp] = sum_s exp(L_end - L_s) c_s u_s k_s^T, and the chunk's L_end.
 // Block: chunk x head x (64 value channels, 128 key channels); a warp takes 16 value channels.
+template <int KT>                        // key channels of a block
 __global__ void __launch_bounds__(128)
 decay_chunk_state_kernel(const __nv_bfloat16 *k, const __nv_bfloat16 *u, const float *la, int la_stride, const float *step,
                          const int32_t *chunk_t0, const int32_t *chunk_n, float *dS, float *l_end, int H, int Hq, int dp, int dvp)
 {
     pdl_wait();
-    extern __shared__ __align__(16) uint8_t ds_smem[];
-    __nv_bfloat16 *us = (__nv_bfloat16 *)ds_smem;                            // [CH][DVT + 8]
-    __nv_bfloat16 *ks = us + DS_CH * (DS_DVT + 8);                           // [CH][kt + 8]
+    __shared__ __align__(16) __nv_bfloat16 us[DS_CH * (DS_DVT + 8)], ks[DS_CH * (KT + 8)];
     __shared__ float Ls[DS_CH], cs[DS_CH];
     const int chunk = blockIdx.x, h = blockIdx.y, hq = h / (H / Hq);
-    const int d_tiles = (dp + DS_DT - 1) / DS_DT;
-    const int v0 = (int)blockIdx.z / d_tiles * DS_DVT, d0 = (int)blockIdx.z % d_tiles * DS_DT;
-    const int vt = min(DS_DVT, dvp - v0), kt = min(DS_DT, dp - d0);
+    const int d_tiles = (dp + KT - 1) / KT;
+    const int v0 = (int)blockIdx.z / d_tiles * DS_DVT, d0 = (int)blockIdx.z % d_tiles * KT;
+    const int vt = min(DS_DVT, dvp - v0), kt = min(KT, dp - d0);
     const int t0 = chunk_t0[chunk], n = chunk_n[chunk];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    // (value channels beyond vt are left as they are in shared memory: their rows of the product are not stored)
-    {
-        const int per = vt / 8;
-        for (int idx = threadIdx.x; idx < DS_CH * per; idx += 128) {
-            const int r = idx / per, c = (idx - r * per) * 8;
-            __nv_bfloat16 *dst = us + r * (DS_DVT + 8) + c;
-            if (r < n) cp16(dst, u + ((size_t)(t0 + r) * H + h) * dvp + v0 + c);
-            else *(uint4 *)dst = make_uint4(0, 0, 0, 0);
-        }
-    }
-    stage_rows(ks, k + ((size_t)t0 * Hq + hq) * dp + d0, (size_t)Hq * dp, n, DS_CH, kt);
-    chunk_decays(la, la_stride, step, H, h, t0, n, Ls, cs);
+    ChunkDecays dec;
+    if (warp == 0) dec.fetch(la, la_stride, step, H, h, t0, n);
+    stage_rows<DS_DVT>(us, u + ((size_t)t0 * H + h) * dvp + v0, (size_t)H * dvp, n, DS_CH, vt);
+    stage_rows<KT>(ks, k + ((size_t)t0 * Hq + hq) * dp + d0, (size_t)Hq * dp, n, DS_CH, kt);
+    if (warp == 0) dec.finish(Ls, cs);
     cp_wait_all();
     __syncthreads();
     const float lend = Ls[n - 1];
     if (blockIdx.z == 0 && threadIdx.x == 0) l_end[(size_t)chunk * H + h] = lend;
     if (warp * 16 >= vt) return;
-    float acc[16][4];
+    constexpr int NT = KT / 8, KP = KT + 8;
+    float acc[NT][4];
 #pragma unroll
-    for (int i = 0; i < 16; i++)
+    for (int i = 0; i < NT; i++)
 #pragma unroll
         for (int j = 0; j < 4; j++) acc[i][j] = 0.f;
-    const int kp = kt + 8;
     const uint32_t ua = smem_addr(us) + (((lane & 7) + (lane >> 4) * 8) * (DS_DVT + 8) + warp * 16 + ((lane >> 3) & 1) * 8) * 2;
-    const uint32_t ka = smem_addr(ks) + (((lane & 7) + ((lane >> 3) & 1) * 8) * kp + (lane >> 4) * 8) * 2;
+    const uint32_t ka = smem_addr(ks) + (((lane & 7) + ((lane >> 3) & 1) * 8) * KP + (lane >> 4) * 8) * 2;
 #pragma unroll
     for (int kk = 0; kk < DS_CH / 16; kk++) {
-        if (kk * 16 >= n) break;
         uint32_t raw[4], hi[4], lo[4];
         ldsm4_t(raw, ua + kk * 16 * (DS_DVT + 8) * 2);
         const int ta = kk * 16 + (lane & 3) * 2;
         float wgt[4];                                                        // tokens ta, ta + 1, ta + 8, ta + 9
 #pragma unroll
-        for (int i = 0; i < 4; i++) {
-            const int t = ta + (i & 1) + (i >> 1) * 8;
-            wgt[i] = __expf(lend - Ls[t]) * cs[t];
+        for (int i = 0; i < 2; i++) {
+            const float2 L = *(const float2 *)&Ls[ta + 8 * i], c = *(const float2 *)&cs[ta + 8 * i];
+            wgt[2 * i] = __expf(lend - L.x) * c.x;
+            wgt[2 * i + 1] = __expf(lend - L.y) * c.y;
         }
 #pragma unroll
         for (int i = 0; i < 4; i++) {                                        // registers: (rows, tokens ta..), (rows + 8, ..), (rows, ta + 8..), ..
@@ -500,20 +502,18 @@ decay_chunk_state_kernel(const __nv_bfloat16 *k, const __nv_bfloat16 *u, const f
             split2(f.x * wgt[(i >> 1) * 2], f.y * wgt[(i >> 1) * 2 + 1], hi[i], lo[i]);
         }
 #pragma unroll
-        for (int nt = 0; nt < 8; nt++) {
-            if (nt * 16 < kt) {
-                uint32_t b[4];
-                ldsm4_t(b, ka + (kk * 16 * kp + nt * 16) * 2);
-                mma16816(acc[2 * nt], hi, b[0], b[1]);
-                mma16816(acc[2 * nt], lo, b[0], b[1]);
-                mma16816(acc[2 * nt + 1], hi, b[2], b[3]);
-                mma16816(acc[2 * nt + 1], lo, b[2], b[3]);
-            }
+        for (int nt = 0; nt < NT / 2; nt++) {
+            uint32_t b[4];
+            ldsm4_t(b, ka + (kk * 16 * KP + nt * 16) * 2);
+            mma16816(acc[2 * nt], hi, b[0], b[1]);
+            mma16816(acc[2 * nt + 1], hi, b[2], b[3]);
+            mma16816(acc[2 * nt], lo, b[0], b[1]);
+            mma16816(acc[2 * nt + 1], lo, b[2], b[3]);
         }
     }
     float *out = dS + (((size_t)chunk * H + h) * dvp + v0 + warp * 16 + (lane >> 2)) * dp + d0 + (lane & 3) * 2;
 #pragma unroll
-    for (int nt = 0; nt < 16; nt++) {
+    for (int nt = 0; nt < NT; nt++) {
         if (nt * 8 < kt) {
             *(float2 *)(out + nt * 8) = make_float2(acc[nt][0], acc[nt][1]);
             *(float2 *)(out + (size_t)8 * dp + nt * 8) = make_float2(acc[nt][2], acc[nt][3]);
@@ -578,8 +578,7 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
 {
     pdl_wait();
     extern __shared__ __align__(16) uint8_t ds_smem[];
-    const int P = dp + 8;
-    const int stage_elems = 2 * DS_DVT * P + DS_CH * (DS_DVT + 8);
+    constexpr int D = NK * 16, P = D + 8, STAGE = 2 * DS_DVT * P + DS_CH * (DS_DVT + 8);
     __nv_bfloat16 *ks = (__nv_bfloat16 *)ds_smem;                            // [CH][P]
     __nv_bfloat16 *stages = ks + DS_CH * P;                                  // per stage: sh, sl [DVT][P], us [CH][DVT + 8]
     __shared__ float Ls[2][DS_CH], cs[2][DS_CH];
@@ -587,40 +586,38 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
     const int hq = blockIdx.y / shares, i0 = (blockIdx.y % shares) * per_block, i1 = min(items, i0 + per_block);
     const int t0 = chunk_t0[chunk], n = chunk_n[chunk];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    ChunkDecays dec;                                                         // (the first warp's, fetched an item ahead)
 
     auto issue = [&](int item, int stage) {
         const int h = hq * rep + item / v_tiles, v0 = item % v_tiles * DS_DVT, vt = min(DS_DVT, dvp - v0);
-        __nv_bfloat16 *sh = stages + stage * stage_elems, *sl = sh + DS_DVT * P, *us = sl + DS_DVT * P;
+        __nv_bfloat16 *sh = stages + stage * STAGE, *sl = sh + DS_DVT * P, *us = sl + DS_DVT * P;
         const __nv_bfloat16 *sp = start + ((size_t)chunk * H + h) * 2 * dvp * dp + (size_t)v0 * dp;
-        stage_rows(sh, sp, dp, vt, vt, dp);
-        stage_rows(sl, sp + (size_t)dvp * dp, dp, vt, vt, dp);
-        const int per = vt / 8;
-        for (int idx = threadIdx.x; idx < DS_CH * per; idx += 128) {
-            const int r = idx / per, c = (idx - r * per) * 8;
-            __nv_bfloat16 *dst = us + r * (DS_DVT + 8) + c;
-            if (r < n) cp16(dst, u + ((size_t)(t0 + r) * H + h) * dvp + v0 + c);
-            else *(uint4 *)dst = make_uint4(0, 0, 0, 0);
-        }
+        stage_rows<D>(sh, sp, dp, vt, DS_DVT, dp);
+        stage_rows<D>(sl, sp + (size_t)dvp * dp, dp, vt, DS_DVT, dp);
+        stage_rows<DS_DVT>(us, u + ((size_t)t0 * H + h) * dvp + v0, (size_t)H * dvp, n, DS_CH, vt);
         asm volatile("cp.async.commit_group;" ::: "memory");
-        chunk_decays(la, la_stride, step, H, h, t0, n, Ls[stage], cs[stage]);        // (the first warp, which has the least to do)
+        if (warp == 0) {
+            dec.finish(Ls[stage], cs[stage]);
+            if (item + 1 < i1) dec.fetch(la, la_stride, step, H, hq * rep + (item + 1) / v_tiles, t0, n);
+        }
     };
-    stage_rows(ks, k + ((size_t)t0 * Hq + hq) * dp, (size_t)Hq * dp, n, DS_CH, dp);
-    issue(i0, 0);
+    if (warp == 0) dec.fetch(la, la_stride, step, H, hq * rep + i0 / v_tiles, t0, n);
+    stage_rows<D>(ks, k + ((size_t)t0 * Hq + hq) * dp, (size_t)Hq * dp, n, DS_CH, dp);
     const int r0 = warp * 16 + (lane >> 2), r1 = r0 + 8;                    // this thread's two tokens
-    const int nkk = dp / 16;
     uint32_t qf[NK][4];
     {
         const __nv_bfloat16 *q0 = q + ((size_t)(t0 + min(r0, n - 1)) * Hq + hq) * dp + (lane & 3) * 2;
         const __nv_bfloat16 *q1 = q + ((size_t)(t0 + min(r1, n - 1)) * Hq + hq) * dp + (lane & 3) * 2;
 #pragma unroll
         for (int kk = 0; kk < NK; kk++) {
-            const bool in = kk < nkk;
+            const bool in = kk * 16 < dp;
             qf[kk][0] = in ? *(const uint32_t *)(q0 + kk * 16) : 0u;
             qf[kk][1] = in ? *(const uint32_t *)(q1 + kk * 16) : 0u;
             qf[kk][2] = in ? *(const uint32_t *)(q0 + kk * 16 + 8) : 0u;
             qf[kk][3] = in ? *(const uint32_t *)(q1 + kk * 16 + 8) : 0u;
         }
     }
+    issue(i0, 0);
     const uint32_t nk = (((lane & 7) + (lane >> 4) * 8) * P + ((lane >> 3) & 1) * 8) * 2;      // [n][k] operands
     const uint32_t ka = smem_addr(ks) + nk;
     const bool works = warp * 16 < n;
@@ -645,18 +642,16 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
                     if (kt <= warp) {
 #pragma unroll
                         for (int kk = 0; kk < NK; kk++) {
-                            if (kk < nkk) {
-                                uint32_t b[4];
-                                ldsm4(b, ka + kt * 16 * P * 2 + kk * 32);
-                                mma16816(s[2 * kt], qf[kk], b[0], b[1]);
-                                mma16816(s[2 * kt + 1], qf[kk], b[2], b[3]);
-                            }
+                            uint32_t b[4];
+                            ldsm4(b, ka + kt * 16 * P * 2 + kk * 32);
+                            mma16816(s[2 * kt], qf[kk], b[0], b[1]);
+                            mma16816(s[2 * kt + 1], qf[kk], b[2], b[3]);
                         }
                     }
                 }
             }
             const int h = hq * rep + item / v_tiles, v0 = item % v_tiles * DS_DVT, vt = min(DS_DVT, dvp - v0);
-            const __nv_bfloat16 *sh = stages + stage * stage_elems, *sl = sh + DS_DVT * P, *us = sl + DS_DVT * P;
+            const __nv_bfloat16 *sh = stages + stage * STAGE, *sl = sh + DS_DVT * P, *us = sl + DS_DVT * P;
             const uint32_t ha = smem_addr(sh) + nk, lo_a = smem_addr(sl) + nk;
             const uint32_t ua = smem_addr(us) + (((lane & 7) + ((lane >> 3) & 1) * 8) * (DS_DVT + 8) + (lane >> 4) * 8) * 2;
             const float dsk = skip ? skip[h] : 0.f;
@@ -668,19 +663,20 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
             // what the state at the chunk's start gives
 #pragma unroll
             for (int kk = 0; kk < NK; kk++) {
-                if (kk < nkk) {
+                uint32_t b[4][4];
 #pragma unroll
-                    for (int nt = 0; nt < 4; nt++) {
-                        if (nt * 16 < vt) {
-                            uint32_t b[4], c[4];
-                            ldsm4(b, ha + nt * 16 * P * 2 + kk * 32);
-                            ldsm4(c, lo_a + nt * 16 * P * 2 + kk * 32);
-                            mma16816(acc[2 * nt], qf[kk], b[0], b[1]);
-                            mma16816(acc[2 * nt + 1], qf[kk], b[2], b[3]);
-                            mma16816(acc[2 * nt], qf[kk], c[0], c[1]);
-                            mma16816(acc[2 * nt + 1], qf[kk], c[2], c[3]);
-                        }
-                    }
+                for (int nt = 0; nt < 4; nt++) ldsm4(b[nt], ha + nt * 16 * P * 2 + kk * 32);
+#pragma unroll
+                for (int nt = 0; nt < 4; nt++) {
+                    mma16816(acc[2 * nt], qf[kk], b[nt][0], b[nt][1]);
+                    mma16816(acc[2 * nt + 1], qf[kk], b[nt][2], b[nt][3]);
+                }
+#pragma unroll
+                for (int nt = 0; nt < 4; nt++) ldsm4(b[nt], lo_a + nt * 16 * P * 2 + kk * 32);
+#pragma unroll
+                for (int nt = 0; nt < 4; nt++) {
+                    mma16816(acc[2 * nt], qf[kk], b[nt][0], b[nt][1]);
+                    mma16816(acc[2 * nt + 1], qf[kk], b[nt][2], b[nt][3]);
                 }
             }
             const float L0 = Ls[stage][r0], L1 = Ls[stage][r1];
@@ -712,14 +708,12 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
                     }
 #pragma unroll
                     for (int nt = 0; nt < 4; nt++) {
-                        if (nt * 16 < vt) {
-                            uint32_t b[4];
-                            ldsm4_t(b, ua + (kt * 16 * (DS_DVT + 8) + nt * 16) * 2);
-                            mma16816(acc[2 * nt], hi, b[0], b[1]);
-                            mma16816(acc[2 * nt + 1], hi, b[2], b[3]);
-                            mma16816(acc[2 * nt], lo, b[0], b[1]);
-                            mma16816(acc[2 * nt + 1], lo, b[2], b[3]);
-                        }
+                        uint32_t b[4];
+                        ldsm4_t(b, ua + (kt * 16 * (DS_DVT + 8) + nt * 16) * 2);
+                        mma16816(acc[2 * nt], hi, b[0], b[1]);
+                        mma16816(acc[2 * nt + 1], hi, b[2], b[3]);
+                        mma16816(acc[2 * nt], lo, b[0], b[1]);
+                        mma16816(acc[2 * nt + 1], lo, b[2], b[3]);
                     }
                 }
             }
@@ -946,15 +940,17 @@ extern "C" int hfb_decay_chunks(const void *q, const void *k, const void *u, con
     float *dS = (float *)scratch;
     __nv_bfloat16 *start = (__nv_bfloat16 *)(dS + (size_t)chunks * st);
     float *l_end = (float *)(start + (size_t)chunks * st * 2);
-    const int v_tiles = (dvp + DS_DVT - 1) / DS_DVT, d_tiles = (dp + DS_DT - 1) / DS_DT;
-    const size_t smem_a = ((size_t)DS_CH * (DS_DVT + 8) + (size_t)DS_CH * ((dp < DS_DT ? dp : DS_DT) + 8)) * 2;
-    g_launch_err = launch_pdl(decay_chunk_state_kernel, dim3(chunks, H, v_tiles * d_tiles), dim3(128), smem_a, (cudaStream_t)s,
-                              (const __nv_bfloat16 *)k, (const __nv_bfloat16 *)u, la, la_stride, step, chunk_t0, chunk_n, dS, l_end, H, Hq, dp, dvp);
+    const int v_tiles = (dvp + DS_DVT - 1) / DS_DVT;
+#define HFB_CHUNK_STATE(KT) \
+    g_launch_err = launch_pdl(decay_chunk_state_kernel<KT>, dim3(chunks, H, v_tiles * ((dp + KT - 1) / KT)), dim3(128), 0, (cudaStream_t)s, \
+                              (const __nv_bfloat16 *)k, (const __nv_bfloat16 *)u, la, la_stride, step, chunk_t0, chunk_n, dS, l_end, H, Hq, dp, dvp)
+    if (dp <= 64) HFB_CHUNK_STATE(64);
+    else HFB_CHUNK_STATE(128);
+#undef HFB_CHUNK_STATE
     if ((rc = check_pdl_launch(g_launch_err, "decay_chunk_state")) != HFB_OK) return rc;
     g_launch_err = launch_pdl(decay_chunk_pass_kernel, dim3((unsigned)((st / 4 + 255) / 256), S), dim3(256), 0, (cudaStream_t)s, dS, l_end, state,
                               (size_t)slot_stride, chunk_first, seq_slots, n_slots, start, H, dp, dvp, error_word());
     if ((rc = check_pdl_launch(g_launch_err, "decay_chunk_pass")) != HFB_OK) return rc;
-    const size_t smem_c = ((size_t)DS_CH * (dp + 8) + 2 * ((size_t)2 * DS_DVT * (dp + 8) + (size_t)DS_CH * (DS_DVT + 8))) * 2;
     // a block's share of the items that read one query/key head: as many as leave four blocks for every SM
     const int items = H / Hq * v_tiles;
     int per_block = items < 8 ? items : 8;
@@ -962,11 +958,11 @@ extern "C" int hfb_decay_chunks(const void *q, const void *k, const void *u, con
     const int shares = (items + per_block - 1) / per_block;
     if ((long)Hq * shares > 65535) return fail(HFB_ENOTSUP, "decay_chunks: %d heads exceed the grid limit", H);
 #define HFB_CHUNK_OUT(NK) do { \
+        const int smem_c = (DS_CH * (NK * 16 + 8) + 2 * (2 * DS_DVT * (NK * 16 + 8) + DS_CH * (DS_DVT + 8))) * 2; \
         static bool opted[64] = {false}; \
         const int dev = current_device(); \
         if (!opted[dev]) { \
-            const int most = (DS_CH * (NK * 16 + 8) + 2 * (2 * DS_DVT * (NK * 16 + 8) + DS_CH * (DS_DVT + 8))) * 2; \
-            cudaError_t e = cudaFuncSetAttribute(decay_chunk_out_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, most); \
+            cudaError_t e = cudaFuncSetAttribute(decay_chunk_out_kernel<NK>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem_c); \
             if (e != cudaSuccess) return fail(HFB_ECUDA, "decay_chunks: %s", cudaGetErrorString(e)); \
             opted[dev] = true; \
         } \

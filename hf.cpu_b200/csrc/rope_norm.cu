@@ -136,7 +136,7 @@ rope_norm_kv_kernel(const float *src, int splits, const void *bias, int bias_dt,
 // [T, QD], keys and values to the token's cache slot (KD = VD = 0: the layer reads another layer's cache), gates as
 // sigmoid(row) to gate_out [T, n_gate] float32.  One block per token.
 template <typename TO>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(1024)
 row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_w, const float *k_w, float eps, const int32_t *slots,
                    TO *q_out, TO *k_cache, TO *v_cache, long long cache_slots, float *gate_out, int n_gate, int T, int QD, int KD, int VD,
                    int vec, int *err)
@@ -144,44 +144,44 @@ row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_
     pdl_entry();
     pdl_sync_small();
     extern __shared__ __align__(16) float rn_row[];                      // [QD + KD]
-    __shared__ float red[16];
-    const int t = blockIdx.x, n = QD + KD;
+    __shared__ float red[64];
+    const int t = blockIdx.x, n = QD + KD, nth = blockDim.x;
     const size_t plane = (size_t)T * row_stride;
     const float *row = src + (size_t)t * row_stride;
     long long slot = (KD + VD > 0 && slots) ? slots[t] : -1;
     if (slot >= cache_slots) { if (threadIdx.x == 0) atomicOr(err, HFB_ERR_SLOT); slot = -1; }
     float sq = 0.f, sk = 0.f;
     if (vec) {
-        for (int c = threadIdx.x * 4; c < n; c += 1024) {
+        for (int c = threadIdx.x * 4; c < n; c += 4 * nth) {
             const float4 v = plane_sum4(row + c, splits, plane);
             *(float4 *)(rn_row + c) = v;
             const float ss = (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
             if (c < QD) sq += ss; else sk += ss;
         }
         if (slot >= 0)
-            for (int c = threadIdx.x * 4; c < VD; c += 1024) store4(v_cache + (size_t)slot * VD + c, plane_sum4(row + n + c, splits, plane));
+            for (int c = threadIdx.x * 4; c < VD; c += 4 * nth) store4(v_cache + (size_t)slot * VD + c, plane_sum4(row + n + c, splits, plane));
     } else {
-        for (int c = threadIdx.x; c < n; c += 256) {
+        for (int c = threadIdx.x; c < n; c += nth) {
             const float v = plane_sum(row + c, splits, plane);
             rn_row[c] = v;
             if (c < QD) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
         }
         if (slot >= 0)
-            for (int c = threadIdx.x; c < VD; c += 256) v_cache[(size_t)slot * VD + c] = from_f32<TO>(plane_sum(row + n + c, splits, plane));
+            for (int c = threadIdx.x; c < VD; c += nth) v_cache[(size_t)slot * VD + c] = from_f32<TO>(plane_sum(row + n + c, splits, plane));
     }
-    for (int c = threadIdx.x; c < n_gate; c += 256)
+    for (int c = threadIdx.x; c < n_gate; c += nth)
         gate_out[(size_t)t * n_gate + c] = 1.0f / (1.0f + expf(-plane_sum(row + n + VD + c, splits, plane)));
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    if (lane == 0) { red[warp] = sq; red[8 + warp] = sk; }
+    if (lane == 0) { red[warp] = sq; red[32 + warp] = sk; }
     __syncthreads();
-    sq = warp_sum(lane < 8 ? red[lane] : 0.f);
-    sk = warp_sum(lane < 8 ? red[8 + lane] : 0.f);
+    sq = warp_sum(lane < nth / 32 ? red[lane] : 0.f);
+    sk = warp_sum(lane < nth / 32 ? red[32 + lane] : 0.f);
     const float rq = 1.0f / sqrtf(sq / (float)QD + eps), rk = 1.0f / sqrtf(sk / (float)max(KD, 1) + eps);
     TO *qo = q_out + (size_t)t * QD, *ko = k_cache + (size_t)(slot < 0 ? 0 : slot) * KD;
     if (vec) {
-        for (int c = threadIdx.x * 4; c < n; c += 1024) {
+        for (int c = threadIdx.x * 4; c < n; c += 4 * nth) {
             const bool is_q = c < QD;
             if (!is_q && slot < 0) continue;
             const float4 w = *(const float4 *)(is_q ? q_w + c : k_w + (c - QD));
@@ -191,7 +191,7 @@ row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_
             store4(is_q ? qo + c : ko + (c - QD), v);
         }
     } else {
-        for (int c = threadIdx.x; c < n; c += 256) {
+        for (int c = threadIdx.x; c < n; c += nth) {
             if (c < QD) qo[c] = from_f32<TO>(rn_row[c] * rq * q_w[c]);
             else if (slot >= 0) ko[c - QD] = from_f32<TO>(rn_row[c] * rk * k_w[c - QD]);
         }
@@ -243,12 +243,15 @@ extern "C" int hfb_row_norm_kv_write(const float *src, int splits, int row_strid
     auto al = [](const void *p, int b) { return ((uintptr_t)p & (b - 1)) == 0; };
     const int vec = ((QD | KD | VD | row_stride) & 3) == 0 && al(src, 16) && al(q_w, 16) && al(k_w, 16) && al(q_out, 4 * esz) &&
                     al(k_cache, 4 * esz) && al(v_cache, 4 * esz);
+    // few rows: what they cost is latency, so as many reads at once as a block has threads for
+    int threads = T <= 128 ? ((QD + KD + 3) / 4 + 31) / 32 * 32 : 256;
+    threads = threads < 256 ? 256 : (threads > 1024 ? 1024 : threads);
 #define HFB_RNK(TY) do { \
         if (smem > 48 * 1024) { \
             cudaError_t e = cudaFuncSetAttribute(row_norm_kv_kernel<TY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return fail(HFB_ECUDA, "row_norm_kv_write: %s", cudaGetErrorString(e)); \
         } \
-        g_launch_err = launch_pdl(row_norm_kv_kernel<TY>, dim3(T), dim3(256), smem, (cudaStream_t)s, src, splits, row_stride, q_w, k_w, eps, slots, \
+        g_launch_err = launch_pdl(row_norm_kv_kernel<TY>, dim3(T), dim3(threads), smem, (cudaStream_t)s, src, splits, row_stride, q_w, k_w, eps, slots, \
             (TY *)q_out, (TY *)k_cache, (TY *)v_cache, (long long)cache_slots, gate_out, n_gate, T, QD, KD, VD, vec, error_word()); \
     } while (0)
     if (out_dt == HFB_F32) HFB_RNK(float);
