@@ -135,8 +135,8 @@ rope_norm_kv_kernel(const float *src, int splits, const void *bias, int bias_dt,
 // `splits` planes.  q = row / sqrt(mean(row^2) + eps) * q_w over the QD queries, keys likewise with k_w; queries to q_out
 // [T, QD], keys and values to the token's cache slot (KD = VD = 0: the layer reads another layer's cache), gates as
 // sigmoid(row) to gate_out [T, n_gate] float32.  One block per token.
-template <typename TO>
-__global__ void __launch_bounds__(1024)
+template <typename TO, int NTH>
+__global__ void __launch_bounds__(NTH)
 row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_w, const float *k_w, float eps, const int32_t *slots,
                    TO *q_out, TO *k_cache, TO *v_cache, long long cache_slots, float *gate_out, int n_gate, int T, int QD, int KD, int VD,
                    int vec, int *err)
@@ -145,7 +145,8 @@ row_norm_kv_kernel(const float *src, int splits, int row_stride, const float *q_
     pdl_sync_small();
     extern __shared__ __align__(16) float rn_row[];                      // [QD + KD]
     __shared__ float red[64];
-    const int t = blockIdx.x, n = QD + KD, nth = blockDim.x;
+    const int t = blockIdx.x, n = QD + KD;
+    constexpr int nth = NTH;
     const size_t plane = (size_t)T * row_stride;
     const float *row = src + (size_t)t * row_stride;
     long long slot = (KD + VD > 0 && slots) ? slots[t] : -1;
@@ -244,18 +245,17 @@ extern "C" int hfb_row_norm_kv_write(const float *src, int splits, int row_strid
     const int vec = ((QD | KD | VD | row_stride) & 3) == 0 && al(src, 16) && al(q_w, 16) && al(k_w, 16) && al(q_out, 4 * esz) &&
                     al(k_cache, 4 * esz) && al(v_cache, 4 * esz);
     // few rows: what they cost is latency, so as many reads at once as a block has threads for
-    int threads = T <= 128 ? ((QD + KD + 3) / 4 + 31) / 32 * 32 : 256;
-    threads = threads < 256 ? 256 : (threads > 1024 ? 1024 : threads);
-#define HFB_RNK(TY) do { \
+#define HFB_RNK(TY, NTH) do { \
         if (smem > 48 * 1024) { \
-            cudaError_t e = cudaFuncSetAttribute(row_norm_kv_kernel<TY>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(row_norm_kv_kernel<TY, NTH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return fail(HFB_ECUDA, "row_norm_kv_write: %s", cudaGetErrorString(e)); \
         } \
-        g_launch_err = launch_pdl(row_norm_kv_kernel<TY>, dim3(T), dim3(threads), smem, (cudaStream_t)s, src, splits, row_stride, q_w, k_w, eps, slots, \
+        g_launch_err = launch_pdl(row_norm_kv_kernel<TY, NTH>, dim3(T), dim3(NTH), smem, (cudaStream_t)s, src, splits, row_stride, q_w, k_w, eps, slots, \
             (TY *)q_out, (TY *)k_cache, (TY *)v_cache, (long long)cache_slots, gate_out, n_gate, T, QD, KD, VD, vec, error_word()); \
     } while (0)
-    if (out_dt == HFB_F32) HFB_RNK(float);
-    else HFB_RNK(__nv_bfloat16);
+    const bool wide = T <= 128 && QD + KD > 1024;
+    if (out_dt == HFB_F32) { if (wide) HFB_RNK(float, 1024); else HFB_RNK(float, 256); }
+    else { if (wide) HFB_RNK(__nv_bfloat16, 1024); else HFB_RNK(__nv_bfloat16, 256); }
 #undef HFB_RNK
     return check_pdl_launch(g_launch_err, "row_norm_kv_write");
 }
