@@ -951,10 +951,15 @@ extern "C" int hfb_decay_chunks(const void *q, const void *k, const void *u, con
     g_launch_err = launch_pdl(decay_chunk_pass_kernel, dim3((unsigned)((st / 4 + 255) / 256), S), dim3(256), 0, (cudaStream_t)s, dS, l_end, state,
                               (size_t)slot_stride, chunk_first, seq_slots, n_slots, start, H, dp, dvp, error_word());
     if ((rc = check_pdl_launch(g_launch_err, "decay_chunk_pass")) != HFB_OK) return rc;
-    // a block's share of the items that read one query/key head: as many as leave four blocks for every SM
-    const int items = H / Hq * v_tiles;
-    int per_block = items < 8 ? items : 8;
-    while (per_block > 1 && (long)chunks * Hq * ((items + per_block - 1) / per_block) < 148 * 4) per_block--;
+    // a block's share of the items that read one query/key head: the one with the fewest rounds over the SMs, a block's start
+    // (keys, queries, the first item's state) counted as one item more
+    const int items = H / Hq * v_tiles, resident = 148 * (dp <= 128 ? 2 : 1);
+    int per_block = 1;
+    long best = -1;
+    for (int p = 1; p <= items && p <= 32; p++) {
+        const long blocks = (long)chunks * Hq * ((items + p - 1) / p), cost = (blocks + resident - 1) / resident * (p + 1);
+        if (best < 0 || cost < best) { best = cost; per_block = p; }
+    }
     const int shares = (items + per_block - 1) / per_block;
     if ((long)Hq * shares > 65535) return fail(HFB_ENOTSUP, "decay_chunks: %d heads exceed the grid limit", H);
 #define HFB_CHUNK_OUT(NK) do { \
