@@ -209,3 +209,19 @@ def test_the_clamps_and_the_window_matter():
         d = copy.deepcopy(c)
         edit(d)
         assert np.abs(plain.forward(d, W, ids) - base).max() > 0.01 * np.abs(base).max()
+
+
+def test_a_model_without_attention_keeps_no_pages(tmp_path, emu):
+    """Only recurrent layers: no cache group at all, the requests' lengths still advance the rotation."""
+    import hfcpu_b200
+    cfg = model(60, 24, 1e-5, 10.0, [layer(ret(8, 8, (0.9, 0.99), 4, 50.0), 16, 0.3), layer(m2(2, 8, 4, 1, 3, 2), 16, 0.3)])
+    folder = make_folder(cfg, str(tmp_path), 5)
+    reqs = requests(60, [30, 7, 12], seed=3)
+    steps = traces.mixed(reqs, max_live=2, prefill_sizes=(5, 2, 9))
+    m = hfcpu_b200.load_model(folder, torch.float32, "cpu")
+    eng = hfcpu_b200.Engine(m, block_size=8, max_tokens=64, max_requests=2)
+    assert eng.cache.groups == []
+    got = traces.run_in_process(eng, steps, check=eng.cache.check)
+    for (r, pos), row in got.items():
+        want = plain_logits(folder, reqs[r])[pos]
+        assert float((row.double() - want).abs().max() / want.abs().max()) < 2e-4, (r, pos)
