@@ -8,8 +8,9 @@ from .peludra import PeludraConfig
 from .mokisun import MokisunConfig
 from .silupel import SilupelConfig
 from .tupalorn import TupalornConfig
+from .birizen import BirizenConfig
 
 __all__ = ["ConfigError", "UnsupportedError", "ModelConfig", "ModelPlan", "PartSpec", "LayerSpec",
            "ScheduleEntry", "Qwen2Config", "ManapelConfig", "PeludraConfig", "MokisunConfig", "SilupelConfig",
-           "TupalornConfig", "config_from_dict", "config_from_gguf", "load_config",
+           "TupalornConfig", "BirizenConfig", "config_from_dict", "config_from_gguf", "load_config",
            "register_architecture", "unregister_architecture", "known_architectures"]

@@ -15,7 +15,7 @@ import dataclasses
 import json
 import os
 from dataclasses import dataclass, field
-from typing import Any, ClassVar, Dict, List, Optional
+from typing import Any, ClassVar, Dict, List, Optional, Tuple
 
 
 class ConfigError(ValueError):
@@ -57,9 +57,12 @@ class ScheduleEntry:
     ``layer`` indexes ``ModelPlan.layers`` (a layer may appear more than once).
     ``cache_of`` names an *earlier entry* whose cache this entry's mixer reads
     instead of keeping one of its own; ``None`` means the entry owns its cache.
+    ``enter`` = (name of one of ``ModelPlan.transitions``, number of the pass): what is done to the stream right in
+    front of this entry.
     """
     layer: int
     cache_of: Optional[int] = None
+    enter: Optional[Tuple[str, int]] = None
 
 
 @dataclass(frozen=True)
@@ -75,6 +78,7 @@ class ModelPlan:
     head: PartSpec
     eos_token_ids: List[int] = field(default_factory=list)
     streams: int = 1                        # copies of the residual stream (hyper-connections); 1: the plain stream
+    transitions: Dict[str, PartSpec] = field(default_factory=dict)     # steps between layers, by name (``ScheduleEntry.enter``)
 
     def validate(self) -> None:
         for i, e in enumerate(self.schedule):
@@ -87,6 +91,11 @@ class ModelPlan:
                 if self.schedule[e.cache_of].cache_of is not None:
                     raise ConfigError(f"schedule entry {i} reads the cache of entry {e.cache_of}, "
                                       f"which has none of its own")
+            if e.enter is not None:
+                if e.enter[0] not in self.transitions:
+                    raise ConfigError(f"schedule entry {i} names transition '{e.enter[0]}', which the plan does not define")
+                if self.streams > 1:
+                    raise UnsupportedError("a transition in front of a layer works on a stream in one copy")
 
 
 @dataclass

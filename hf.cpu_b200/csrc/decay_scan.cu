@@ -57,14 +57,31 @@ template <typename TO> __device__ __forceinline__ float silu_for(float z)
     else return __fdividef(z, 1.0f + __expf(-z));
 }
 
+template <typename TO> __device__ __forceinline__ float sigmoid_for(float z)
+{
+    if constexpr (sizeof(TO) == 4) return 1.0f / (1.0f + expf(-z));
+    else return __fdividef(1.0f, 1.0f + __expf(-z));
+}
+
 __device__ __forceinline__ void store2(float *p, float a, float b) { *(float2 *)p = make_float2(a, b); }
 __device__ __forceinline__ void store2(__nv_bfloat16 *p, float a, float b) { *(__nv_bfloat162 *)p = __floats2bfloat162_rn(a, b); }
 
 // ---- operands of retention --------------------------------------------------------------------------------------
+template <typename TO, bool SILU> __device__ __forceinline__ float head_in(const float *p, int splits, size_t plane)
+{
+    const float v = plane_sum(p, splits, plane);
+    return SILU ? silu_for<TO>(v) : v;
+}
+template <typename TO, bool SILU> __device__ __forceinline__ float2 head_in2(const float *p, int splits, size_t plane)
+{
+    const float2 v = plane_sum2(p, splits, plane);
+    return SILU ? make_float2(silu_for<TO>(v.x), silu_for<TO>(v.y)) : v;
+}
+
 // One warp per (token, head) of the rows [H query heads of d | H key heads of d | H value heads of dv | ...] (row_stride
 // floats, `splits` planes): rotation of the first n_rot dimensions of queries and keys (pairs i, i + n_rot/2), keys times
-// k_scale, everything to its padded place.
-template <typename TO>
+// k_scale, everything to its padded place.  SILU: queries, keys and values pass silu first.
+template <typename TO, bool SILU>
 __global__ void __launch_bounds__(128)
 rotate_heads_kernel(const float *src, int splits, int row_stride, const float *cos_sin, int n_rot, int n_positions,
                     const int32_t *positions, float k_scale, TO *q, TO *k, TO *u, int T, int H, int d, int dv, int dp, int dvp, int pairs,
@@ -90,8 +107,8 @@ rotate_heads_kernel(const float *src, int splits, int row_stride, const float *c
         // two neighbouring dimensions a lane: everything of the head is even and aligned to two
         for (int i = 2 * lane; i < half; i += 64) {
             const float4 c = *(const float4 *)(cs + 2 * i);
-            const float2 qa = plane_sum2(qr + i, splits, plane), qb = plane_sum2(qr + i + half, splits, plane);
-            const float2 ka = plane_sum2(kr + i, splits, plane), kb = plane_sum2(kr + i + half, splits, plane);
+            const float2 qa = head_in2<TO, SILU>(qr + i, splits, plane), qb = head_in2<TO, SILU>(qr + i + half, splits, plane);
+            const float2 ka = head_in2<TO, SILU>(kr + i, splits, plane), kb = head_in2<TO, SILU>(kr + i + half, splits, plane);
             float lo0, hi0, lo1, hi1;
             rope_pair(qa.x, qb.x, c.x, c.y, lo0, hi0);
             rope_pair(qa.y, qb.y, c.z, c.w, lo1, hi1);
@@ -103,13 +120,13 @@ rotate_heads_kernel(const float *src, int splits, int row_stride, const float *c
             store2(kd + i + half, hi0 * k_scale, hi1 * k_scale);
         }
         for (int i = n_rot + 2 * lane; i < dp; i += 64) {
-            const float2 a = i < d ? plane_sum2(qr + i, splits, plane) : make_float2(0.f, 0.f);
-            const float2 b = i < d ? plane_sum2(kr + i, splits, plane) : make_float2(0.f, 0.f);
+            const float2 a = i < d ? head_in2<TO, SILU>(qr + i, splits, plane) : make_float2(0.f, 0.f);
+            const float2 b = i < d ? head_in2<TO, SILU>(kr + i, splits, plane) : make_float2(0.f, 0.f);
             store2(qd + i, a.x, a.y);
             store2(kd + i, b.x * k_scale, b.y * k_scale);
         }
         for (int i = 2 * lane; i < dvp; i += 64) {
-            const float2 a = i < dv ? plane_sum2(vr + i, splits, plane) : make_float2(0.f, 0.f);
+            const float2 a = i < dv ? head_in2<TO, SILU>(vr + i, splits, plane) : make_float2(0.f, 0.f);
             store2(ud + i, a.x, a.y);
         }
         return;
@@ -121,13 +138,13 @@ rotate_heads_kernel(const float *src, int splits, int row_stride, const float *c
         const float f = part ? k_scale : 1.0f;
         for (int i = lane; i < half; i += 32) {
             float lo, hi;
-            rope_pair(plane_sum(p + i, splits, plane), plane_sum(p + i + half, splits, plane), cs[2 * i], cs[2 * i + 1], lo, hi);
+            rope_pair(head_in<TO, SILU>(p + i, splits, plane), head_in<TO, SILU>(p + i + half, splits, plane), cs[2 * i], cs[2 * i + 1], lo, hi);
             dst[i] = from_f32<TO>(lo * f);
             dst[i + half] = from_f32<TO>(hi * f);
         }
-        for (int i = n_rot + lane; i < dp; i += 32) dst[i] = from_f32<TO>(i < d ? plane_sum(p + i, splits, plane) * f : 0.f);
+        for (int i = n_rot + lane; i < dp; i += 32) dst[i] = from_f32<TO>(i < d ? head_in<TO, SILU>(p + i, splits, plane) * f : 0.f);
     }
-    for (int i = lane; i < dvp; i += 32) ud[i] = from_f32<TO>(i < dv ? plane_sum(vr + i, splits, plane) : 0.f);
+    for (int i = lane; i < dvp; i += 32) ud[i] = from_f32<TO>(i < dv ? head_in<TO, SILU>(vr + i, splits, plane) : 0.f);
 }
 
 // ---- operands of the state-space form ---------------------------------------------------------------------------
@@ -739,10 +756,10 @@ decay_chunk_out_kernel(const __nv_bfloat16 *q, const __nv_bfloat16 *k, const __n
 }
 
 // ---- behind the recurrence --------------------------------------------------------------------------------------
-// A row of o [T, C] in parts of n values, each divided by its own root mean square; the gate silu(g) multiplies before the
-// norm (gate_first) or after it; times a weight [C] where there is one.  g is the sum of `splits` planes [T, g_stride] read
+// A row of o [T, C] in parts of n values, each divided by its own root mean square; the gate, silu(g) or (SIGMOID) sigmoid(g),
+// multiplies before the norm (gate_first) or after it; times a weight [C] where there is one.  g is the sum of `splits` planes [T, g_stride] read
 // from column g_col0 on.  TH threads per part, at most 16 values a thread, V at a time.
-template <typename TO, int TH, int V, int N>
+template <typename TO, int TH, int V, int N, bool SIGMOID>
 __global__ void __launch_bounds__(TH < 128 ? 128 : TH)
 part_norm_gate_kernel(const float *o, const float *g, int splits, int g_stride, int g_col0, const float *w, float eps, int gate_first,
                       TO *out, size_t out_stride, int T, int C, int n, int parts)
@@ -776,7 +793,7 @@ part_norm_gate_kernel(const float *o, const float *g, int splits, int g_stride, 
     }
 #pragma unroll
     for (int j = 0; j < N * V; j++) {
-        gate[j] = silu_for<TO>(gate[j]);
+        gate[j] = SIGMOID ? sigmoid_for<TO>(gate[j]) : silu_for<TO>(gate[j]);
         if (gate_first) v[j] *= gate[j];
         ss = fmaf(v[j], v[j], ss);
     }
@@ -823,7 +840,7 @@ static int bad_sizes(const char *who, int H, int Hq, int d, int dv, int dp, int 
 
 extern "C" int hfb_rotate_heads(const float *src, int splits, int row_stride, const float *cos_sin, int n_rot, int n_positions,
                                 const int32_t *positions, float k_scale, void *q, void *k, void *u, int out_dt, int T, int H, int d, int dv,
-                                int dp, int dvp, hfb_stream s)
+                                int dp, int dvp, int silu, hfb_stream s)
 {
     if (T <= 0) return HFB_OK;
     int rc = bad_sizes("rotate_heads", H, H, d, dv, dp, dvp);
@@ -835,13 +852,12 @@ extern "C" int hfb_rotate_heads(const float *src, int splits, int row_stride, co
     // (dp and dvp are multiples of 16, the outputs' heads therefore aligned)
     const int pairs = (d & 1) == 0 && (dv & 1) == 0 && (row_stride & 1) == 0 && (n_rot & 3) == 0 && ((uintptr_t)src & 7) == 0 && aligned16(cos_sin) &&
                       aligned16(q) && aligned16(k) && aligned16(u);
-    if (out_dt == HFB_F32)
-        g_launch_err = launch_pdl(rotate_heads_kernel<float>, grid, dim3(128), 0, (cudaStream_t)s, src, splits, row_stride, cos_sin, n_rot, n_positions,
-                                  positions, k_scale, (float *)q, (float *)k, (float *)u, T, H, d, dv, dp, dvp, pairs, error_word());
-    else
-        g_launch_err = launch_pdl(rotate_heads_kernel<__nv_bfloat16>, grid, dim3(128), 0, (cudaStream_t)s, src, splits, row_stride, cos_sin, n_rot,
-                                  n_positions, positions, k_scale, (__nv_bfloat16 *)q, (__nv_bfloat16 *)k, (__nv_bfloat16 *)u, T, H, d, dv, dp,
-                                  dvp, pairs, error_word());
+#define HFB_ROT(TY, SILU) \
+    g_launch_err = launch_pdl(rotate_heads_kernel<TY, SILU>, grid, dim3(128), 0, (cudaStream_t)s, src, splits, row_stride, cos_sin, n_rot, n_positions, \
+                              positions, k_scale, (TY *)q, (TY *)k, (TY *)u, T, H, d, dv, dp, dvp, pairs, error_word())
+    if (out_dt == HFB_F32) { if (silu) HFB_ROT(float, true); else HFB_ROT(float, false); }
+    else { if (silu) HFB_ROT(__nv_bfloat16, true); else HFB_ROT(__nv_bfloat16, false); }
+#undef HFB_ROT
     return check_pdl_launch(g_launch_err, "rotate_heads");
 }
 
@@ -983,7 +999,8 @@ extern "C" int hfb_decay_chunks(const void *q, const void *k, const void *u, con
 }
 
 extern "C" int hfb_part_norm_gate(const float *o, const float *g, int splits, int g_stride, int g_col0, const float *w, float eps,
-                                  int gate_first, void *out, int out_dt, int64_t out_stride, int T, int C, int parts, hfb_stream s)
+                                  int gate_first, int sigmoid, void *out, int out_dt, int64_t out_stride, int T, int C, int parts,
+                                  hfb_stream s)
 {
     if (T <= 0) return HFB_OK;
     if (!o || !g || splits < 1 || C <= 0 || parts < 1 || C % parts || g_col0 < 0 || g_col0 + C > g_stride || !out || !valid_dt(out_dt) || out_stride < C)
@@ -993,20 +1010,20 @@ extern "C" int hfb_part_norm_gate(const float *o, const float *g, int splits, in
     if (parts > 65535) return fail(HFB_ENOTSUP, "part_norm_gate: %d parts exceed the grid limit", parts);
     const bool vec = (n & 3) == 0 && (g_stride & 3) == 0 && (g_col0 & 3) == 0 && aligned16(o) && aligned16(g) && (out_stride & 3) == 0 &&
                      ((uintptr_t)out & (4 * esz - 1)) == 0;
-#define HFB_PNG(TY, TH, V, N) \
-    g_launch_err = launch_pdl(part_norm_gate_kernel<TY, TH, V, N>, dim3(T, TH < 128 ? (parts + 128 / TH - 1) / (128 / TH) : parts), dim3(TH < 128 ? 128 : TH), \
+#define HFB_PNG(TY, TH, V, N, SG) \
+    g_launch_err = launch_pdl(part_norm_gate_kernel<TY, TH, V, N, SG>, dim3(T, TH < 128 ? (parts + 128 / TH - 1) / (128 / TH) : parts), dim3(TH < 128 ? 128 : TH), \
                               0, (cudaStream_t)s, o, g, splits, g_stride, g_col0, w, eps, gate_first, (TY *)out, (size_t)out_stride, T, C, n, parts)
     // a warp for parts of up to 128, 256 or 512 values, else a block
-#define HFB_PNGT(TY) do { \
+#define HFB_PNGT(TY, SG) do { \
         if (vec) { \
-            if (n <= 128) HFB_PNG(TY, 32, 4, 1); else if (n <= 256) HFB_PNG(TY, 32, 4, 2); else if (n <= 512) HFB_PNG(TY, 32, 4, 4); \
-            else if (n <= 2048) HFB_PNG(TY, 256, 4, 2); else if (n <= 4096) HFB_PNG(TY, 256, 4, 4); else HFB_PNG(TY, 1024, 4, 4); \
+            if (n <= 128) HFB_PNG(TY, 32, 4, 1, SG); else if (n <= 256) HFB_PNG(TY, 32, 4, 2, SG); else if (n <= 512) HFB_PNG(TY, 32, 4, 4, SG); \
+            else if (n <= 2048) HFB_PNG(TY, 256, 4, 2, SG); else if (n <= 4096) HFB_PNG(TY, 256, 4, 4, SG); else HFB_PNG(TY, 1024, 4, 4, SG); \
         } else { \
-            if (n <= 512) HFB_PNG(TY, 32, 1, 16); else if (n <= 4096) HFB_PNG(TY, 256, 1, 16); else HFB_PNG(TY, 1024, 1, 16); \
+            if (n <= 512) HFB_PNG(TY, 32, 1, 16, SG); else if (n <= 4096) HFB_PNG(TY, 256, 1, 16, SG); else HFB_PNG(TY, 1024, 1, 16, SG); \
         } \
     } while (0)
-    if (out_dt == HFB_F32) HFB_PNGT(float);
-    else HFB_PNGT(__nv_bfloat16);
+    if (out_dt == HFB_F32) { if (sigmoid) HFB_PNGT(float, true); else HFB_PNGT(float, false); }
+    else { if (sigmoid) HFB_PNGT(__nv_bfloat16, true); else HFB_PNGT(__nv_bfloat16, false); }
 #undef HFB_PNGT
 #undef HFB_PNG
     return check_pdl_launch(g_launch_err, "part_norm_gate");

@@ -214,6 +214,15 @@ int hfb_dyt_residual(const void *y, int y_dt, int splits, const void *bias, int 
                      float *residual, const void *alpha2, const void *w2, const void *b2, int p2_dt,
                      void *out, int out_dt, int M, int E, hfb_stream s);
 
+/* The tail of a sublayer whose output is normed before it joins the stream, or of a step between layers, one pass over
+ * the rows: v = sum of y's `splits` planes [splits, M, N] (+ bias [N]) (+ sum_j mix_w[m, j] * mix_y[m * top + j, :], float32,
+ * null: none); with post_w [N], v = v / sqrt(mean(v^2) + post_eps) * post_w; residual = (base, or residual where base is
+ * null) + v; with out, out = residual / sqrt(mean(residual^2) + next_eps) * next_w, or residual itself where next_w is null.
+ * splits = 0 without a mix: only out. */
+int hfb_rms_tail(const float *y, int splits, const void *bias, int bias_dt, const float *mix_y, const float *mix_w, int top,
+                 const void *post_w, int post_dt, float post_eps, const float *base, float *residual, const void *next_w,
+                 int next_dt, float next_eps, void *out, int out_dt, int M, int N, hfb_stream s);
+
 /* The tail of a q|k|v product: src [splits, T, H d + G d + G dv] float32 partial sums (+ bias) -> rotation of the first
  * n_rot dimensions of query and key heads -> with norm != 0, x / sqrt(mean(x^2) + eps) per head, times q_w / k_w
  * (float32 [d], shared by the heads; null: no weight) -> q_out [T, H d], keys [.., G, d] and values [.., G, dv] at cache
@@ -230,10 +239,13 @@ int hfb_rope_norm_kv_write(const float *src, int splits, const void *bias, int b
 /* Latent attention, the tail of the down product: src [splits, T, q_rank + kv_rank + rot] float32 partial sums ->
  * query latent = rmsnorm(src[:q_rank]) * q_w -> cq_out [T, q_rank]; key/value latent = rmsnorm(next kv_rank) * kv_w ->
  * cache row [0, kv_rank); the last `rot` values rotated (pairs (2i, 2i+1), cos_sin [n_positions, rot / 2, 2]) -> cache
- * row [kv_rank, kv_rank + rot).  The cache holds one row of kv_rank + rot per slot.  Norm weights float32. */
+ * row [kv_rank, kv_rank + rot).  The cache holds one row of kv_rank + rot per slot.  Norm weights float32.  Rows of src are
+ * row_stride floats; with n_gate > 0 the next n_gate values of a row are an output gate's, whose sigmoids go to gate_out
+ * [T, n_gate]. */
 int hfb_latent_split(const float *src, int splits, const float *q_w, const float *kv_w, float eps, const float *cos_sin,
                      int n_positions, const int32_t *positions, const int32_t *slots, void *cq_out, void *cache,
-                     int out_dt, int64_t cache_slots, int T, int q_rank, int kv_rank, int rot, hfb_stream s);
+                     int out_dt, int64_t cache_slots, int T, int q_rank, int kv_rank, int rot, int row_stride, void *gate_out,
+                     int n_gate, hfb_stream s);
 
 /* Latent attention, the tail of the query product: src [splits, T, H (d + rot)] float32 partial sums; per head the
  * first d values go to q_plain [T, H, d] as they are, the last `rot` rotated (pairs (2i, 2i+1)) to
@@ -250,9 +262,10 @@ int hfb_latent_query_absorb(const float *src, int splits, const float *cos_sin, 
 
 /* A product per head: out[t, h, n] = sum_k w[h, n, k] * in[t, h, k], n < N, k < K; rows of `in` hold H heads in_row
  * apart from column 0, rows of `out` H heads out_row apart (in_row >= K, out_row >= N: a head's result may land in the
- * first N columns of a wider row).  float32 sums; operands all bfloat16 (tensor cores) or all float32. */
+ * first N columns of a wider row).  float32 sums; operands all bfloat16 (tensor cores) or all float32.  gate [T, H * N] in
+ * out's type (null: none): factors on the result. */
 int hfb_headwise_linear(const void *in, int in_dt, const void *w, int w_dt, void *out, int out_dt, int T, int H, int N,
-                        int K, int in_row, int out_row, hfb_stream s);
+                        int K, int in_row, int out_row, const void *gate, hfb_stream s);
 
 /* The choice of a mixture of experts' router from its float32 logits z [splits, T, E] (partial sums of the router's
  * product, summed in order, plus its bias; finished logits: splits = 1, bias null): the `top` largest (lowest index first
@@ -269,20 +282,24 @@ int hfb_moe_sort(const int32_t *ids, int pairs, int E, int tile, int32_t *order,
 
 /* Grouped product over the sorted places: out[dst(p), :] = act(a[src(p), :] . w[expert(p)]^T), w [E, N, K].
  * src(p) = order[p] / src_div when src_div > 0, else p; dst(p) = order[p] when scatter != 0, else p.  `tile`: the most
- * places a tile of the lists holds, up to 128; with 16 and less the form for steps of a few tokens runs. */
-int hfb_moe_gemm(const void *a, int a_dt, const void *w, int w_dt, void *out, int out_dt, int act, int N, int K,
+ * places a tile of the lists holds, up to 128; with 16 and less the form for steps of a few tokens runs.  act may be
+ * HFB_ACT_GLU | HFB_ACT_CLAMPED_GLU with its constants. */
+int hfb_moe_gemm(const void *a, int a_dt, const void *w, int w_dt, void *out, int out_dt, int act, float limit, float alpha,
+                 float offset, int N, int K,
                  const int32_t *order, int src_div, int scatter, const int32_t *tile_expert, const int32_t *tile_p0,
                  const int32_t *tile_n, const int32_t *n_tiles, int max_tiles, int tile, hfb_stream s);
 
 /* out[t, :] = sum_j weights[t, j] * y[t * top + j, :] in float32, j in order */
 int hfb_moe_combine(const void *y, int y_dt, const float *weights, float *out, int T, int top, int N, hfb_stream s);
 
-/* The router of a mixture whose scores are a softmax over all router outputs: z [splits, T, E] float32 partial sums;
- * s = softmax(z); choice score = s + correction (null: none); the outputs form n_groups equal groups of neighbours and
- * only those of the `keep` groups with the largest choice score can be chosen; ids [T, top] = the `top` largest choice
- * scores (largest first, the lower index among equals), weights = s[ids] * scale. */
-int hfb_moe_route_softmax(const float *z, int splits, const void *correction, int corr_dt, int T, int E, int top,
-                          int n_groups, int keep, float scale, int32_t *ids, float *weights, hfb_stream s);
+/* The router of a mixture that scores every output: z [splits, T, E] float32 partial sums; s = softmax(z) over all outputs
+ * (score 0) or sigmoid(z) (score 1); choice score = s + correction (null: none); the outputs form n_groups equal groups of
+ * neighbours, a group counts as much as the sum of its group_best (1 or 2) largest choice scores, and only outputs of the
+ * `keep` best groups can be chosen; ids [T, top] = the `top` largest choice scores (largest first, the lower index among
+ * equals), weights = s[ids], with renorm divided by their sum + 1e-20, times scale. */
+int hfb_moe_route_scored(const float *z, int splits, const void *correction, int corr_dt, int T, int E, int top, int score,
+                         int n_groups, int keep, int group_best, int renorm, float scale, int32_t *ids, float *weights,
+                         hfb_stream s);
 
 /* Hyper-connections: the residual stream in S copies, x [T, S, E] float32.
  * hc_spread: every copy = emb [T, E].
@@ -332,15 +349,16 @@ int hfb_conv_carry(const float *x, int splits, int x_stride, int x_col0, int tap
  * [H][dvp][dp] float32 per slot, q, k [T][heads][dp], u [T][H][dvp] in the run's type, zeros in the padding (dp, dvp: d,
  * dv rounded up to a multiple of 16), o [T][H][dv] float32; la [T][H] (la_stride H) or [H] (la_stride 0), step c [T][H] or
  * NULL (1), skip [H] or NULL (0); head h reads query/key head h / (H / Hq).
- * rotate_heads: q, k, u from rows [H q heads | H k heads | H v heads | ..]: rotation (pairs i, i + n_rot / 2), keys times k_scale.
+ * rotate_heads: q, k, u from rows [H q heads | H k heads | H v heads | ..]: silu of all three (silu != 0), rotation (pairs i,
+ *   i + n_rot / 2), keys times k_scale.
  * state_space_operands: q, k, u, step, la from rows [z: H dv | x: H dv | B: G d | C: G d | dt: H | ..]: x, B, C through a
  *   causal convolution with bias and silu (carried inputs as in conv_carry), step = softplus(dt + dt_bias), la = -rate step.
  * decay_walk: token by token.  decay_chunks: chunks of hfb_decay_chunk_tokens() tokens, bfloat16 operands.
- * part_norm_gate: rows of o in `parts` equal parts, each divided by its root mean square; silu(g) multiplies before
- *   (gate_first) or after; times w [C] where given; rows of out out_stride elements apart. */
+ * part_norm_gate: rows of o in `parts` equal parts, each divided by its root mean square; silu(g), or sigmoid(g) (sigmoid != 0),
+ *   multiplies before (gate_first) or after; times w [C] where given; rows of out out_stride elements apart. */
 int hfb_rotate_heads(const float *src, int splits, int row_stride, const float *cos_sin, int n_rot, int n_positions,
                      const int32_t *positions, float k_scale, void *q, void *k, void *u, int out_dt, int T, int H, int d, int dv,
-                     int dp, int dvp, hfb_stream s);
+                     int dp, int dvp, int silu, hfb_stream s);
 int hfb_state_space_operands(const float *src, int splits, int row_stride, const void *w, int w_dt, const void *bias, int bias_dt,
                              int taps, const void *dt_bias, int dtb_dt, const float *rate, float *carried, int64_t slot_stride,
                              const int32_t *token_seq, const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, int S,
@@ -356,7 +374,7 @@ int hfb_decay_chunks(const void *q, const void *k, const void *u, const float *l
                      const int32_t *chunk_first, int chunks, const int32_t *seq_slots, int n_slots, int S, void *scratch,
                      size_t scratch_bytes, float *o, int H, int Hq, int d, int dv, int dp, int dvp, hfb_stream s);
 int hfb_part_norm_gate(const float *o, const float *g, int splits, int g_stride, int g_col0, const float *w, float eps,
-                       int gate_first, void *out, int out_dt, int64_t out_stride, int T, int C, int parts, hfb_stream s);
+                       int gate_first, int sigmoid, void *out, int out_dt, int64_t out_stride, int T, int C, int parts, hfb_stream s);
 
 /* Attention whose queries and keys are normed over the whole projection: the q|k|v|head gates tail (no rotation), and the
  * gate of one number per head: out[t, h, :] = a[t, h, :] * gate[t, h]. */

@@ -17,12 +17,16 @@ constexpr int LS_MAX_WARPS = 16;
 
 // One block per token: the row [query latent | key/value latent | rotated part] is summed over the product's partial sums
 // into shared memory with 16-byte reads (where the sizes allow), both sums of squares are reduced in one go, and the three
-// parts leave in their forms: two normed and weighted, one rotated in pairs (2i, 2i + 1).
+// parts leave in their forms: two normed and weighted, one rotated in pairs (2i, 2i + 1).  Where the row goes on with the
+// columns of an output gate (n_gate of them; rows are row_stride floats apart), the blocks with blockIdx.y > 0 store their
+// sigmoids, LS_GATE columns each.
+constexpr int LS_GATE = 1024;
+
 template <typename TO>
 __global__ void __launch_bounds__(LS_MAX_WARPS * 32)
 latent_split_kernel(const float *src, int splits, const float *q_w, const float *kv_w, float eps, const float *cos_sin,
                     int n_positions, const int32_t *positions, const int32_t *slots, TO *cq_out, TO *cache,
-                    long long cache_slots, int T, int q_rank, int kv_rank, int rot, int *err)
+                    long long cache_slots, int T, int q_rank, int kv_rank, int rot, int row_stride, TO *gate_out, int n_gate, int *err)
 {
     pdl_entry();
     pdl_sync_small();
@@ -31,10 +35,33 @@ latent_split_kernel(const float *src, int splits, const float *q_w, const float 
     const int threads = blockDim.x, warps = threads >> 5;
     const int t = blockIdx.x;
     const int C = q_rank + kv_rank + rot, kv0 = q_rank, rot0 = q_rank + kv_rank;
-    const size_t plane = (size_t)T * C;
-    const float *p = src + (size_t)t * C;
+    const size_t plane = (size_t)T * row_stride;
+    const float *p = src + (size_t)t * row_stride;
+    if (blockIdx.y > 0) {
+        const int c0 = ((int)blockIdx.y - 1) * LS_GATE, c1 = min(n_gate, c0 + LS_GATE);
+        TO *g = gate_out + (size_t)t * n_gate;
+        const bool vec = ((C | row_stride | n_gate) & 3) == 0 && ((uintptr_t)src & 15) == 0 && ((uintptr_t)gate_out & 15) == 0;
+        if (vec) {
+            for (int c = c0 + threadIdx.x * 4; c < c1; c += threads * 4) {
+                const float4 z = plane_sum4(p + C + c, splits, plane);
+                const float a = 1.0f / (1.0f + expf(-z.x)), b = 1.0f / (1.0f + expf(-z.y));
+                const float d = 1.0f / (1.0f + expf(-z.z)), e = 1.0f / (1.0f + expf(-z.w));
+                if constexpr (sizeof(TO) == 4) {
+                    *(float4 *)(g + c) = make_float4(a, b, d, e);
+                } else {
+                    uint2 u;
+                    u.x = pack_bf16(a, b);
+                    u.y = pack_bf16(d, e);
+                    *(uint2 *)(g + c) = u;
+                }
+            }
+        } else {
+            for (int c = c0 + threadIdx.x; c < c1; c += threads) g[c] = from_f32<TO>(1.0f / (1.0f + expf(-plane_sum(p + C + c, splits, plane))));
+        }
+        return;
+    }
     float ss_q = 0.f, ss_kv = 0.f;
-    const bool vec = ((q_rank | kv_rank | rot) & 3) == 0 && ((uintptr_t)src & 15) == 0;
+    const bool vec = ((q_rank | kv_rank | rot | row_stride) & 3) == 0 && ((uintptr_t)src & 15) == 0;
     if (vec) {
         for (int c = threadIdx.x * 4; c < C; c += threads * 4) {
             float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -130,7 +157,7 @@ constexpr int HW_TT = 16, HW_NT = 64, HW_KC = 32;
 
 template <typename TI, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
-headwise_linear_kernel(const TI *in, const TW *w, TO *out, int T, int H, int N, int K, int in_row, int out_row)
+headwise_linear_kernel(const TI *in, const TW *w, TO *out, int T, int H, int N, int K, int in_row, int out_row, const TO *gate)
 {
     pdl_sync();
     __shared__ float As[HW_TT][HW_KC + 1];
@@ -163,7 +190,9 @@ headwise_linear_kernel(const TI *in, const TW *w, TO *out, int T, int H, int N, 
     if (n < N)
         for (int i = 0; i < 4; i++) {
             const int t = t0 + ty * 4 + i;
-            if (t < T) out[((size_t)t * H + h) * out_row + n] = from_f32<TO>(acc[i]);
+            if (t >= T) continue;
+            const float f = gate ? to_f32(gate[((size_t)t * H + h) * N + n]) : 1.0f;
+            out[((size_t)t * H + h) * out_row + n] = from_f32<TO>(acc[i] * f);
         }
 }
 
@@ -180,7 +209,7 @@ template <int MODE>
 __global__ void __launch_bounds__(128)
 headwise_mma_kernel(const __nv_bfloat16 *in, const float *src, int splits, const __nv_bfloat16 *w, __nv_bfloat16 *out, int T,
                     int H, int N, int K, int in_row, int out_row, const float *cos_sin, int n_positions,
-                    const int32_t *positions, int rot, int att_col, int *err)
+                    const int32_t *positions, int rot, int att_col, const __nv_bfloat16 *gate, int *err)
 {
     __shared__ __align__(16) __nv_bfloat16 As[HM_T][HM_KP];
     __shared__ __align__(16) __nv_bfloat16 Ws[HM_N][HM_KP];
@@ -286,7 +315,12 @@ headwise_mma_kernel(const __nv_bfloat16 *in, const float *src, int splits, const
 #pragma unroll
         for (int nn = 0; nn < 8; nn++) {
             const int n = n0 + nn * 8 + (lane & 3) * 2;
-            const float x = acc[nn][half * 2], y = acc[nn][half * 2 + 1];
+            float x = acc[nn][half * 2], y = acc[nn][half * 2 + 1];
+            if (MODE == 0 && gate) {
+                const __nv_bfloat16 *gp = gate + ((size_t)t * H + h) * N + n;
+                if (n < N) x *= __bfloat162float(gp[0]);
+                if (n + 1 < N) y *= __bfloat162float(gp[1]);
+            }
             if (n + 1 < N && pair_ok) *(uint32_t *)(o + n) = pack_bf16(x, y);
             else {
                 if (n < N) o[n] = __float2bfloat16_rn(x);
@@ -327,27 +361,31 @@ static int headwise_tiles_y(int T, int N, int K) { return (K <= HM_K && T >= 512
 
 extern "C" int hfb_latent_split(const float *src, int splits, const float *q_w, const float *kv_w, float eps, const float *cos_sin,
                                 int n_positions, const int32_t *positions, const int32_t *slots, void *cq_out, void *cache,
-                                int out_dt, int64_t cache_slots, int T, int q_rank, int kv_rank, int rot, hfb_stream s)
+                                int out_dt, int64_t cache_slots, int T, int q_rank, int kv_rank, int rot, int row_stride, void *gate_out,
+                                int n_gate, hfb_stream s)
 {
     if (T <= 0) return HFB_OK;
     if (!valid_dt(out_dt) || splits < 1 || q_rank <= 0 || kv_rank <= 0 || rot < 0 || (rot & 1) || !q_w || !kv_w || !cq_out)
         return fail(HFB_EINVAL, "latent_split: bad arguments (q_rank=%d kv_rank=%d rot=%d)", q_rank, kv_rank, rot);
     if (rot > 0 && (!cos_sin || !positions)) return fail(HFB_EINVAL, "latent_split: rotation needs a table and positions");
     if (slots && !cache) return fail(HFB_EINVAL, "latent_split: the latent rows need a cache");
+    if (n_gate < 0 || (n_gate > 0 && !gate_out) || row_stride < q_rank + kv_rank + rot + n_gate)
+        return fail(HFB_EINVAL, "latent_split: bad row (%d values, %d of them gates)", row_stride, n_gate);
     const size_t smem = (size_t)(q_rank + kv_rank + rot) * sizeof(float);
     if (smem > 40 * 1024) return fail(HFB_ENOTSUP, "latent_split: rows above %d values are not supported", 40 * 1024 / 4);
-    const dim3 grid(T);
+    const dim3 grid(T, 1 + (n_gate + LS_GATE - 1) / LS_GATE);
     // The number of threads goes with the row's width only, never with the number of tokens: the order in which a row's
     // squares are summed must not depend on what else the step holds.
     const int row = q_rank + kv_rank + rot;
     const dim3 block(row >= 2048 ? LS_MAX_WARPS * 32 : (row >= 768 ? 256 : LS_THREADS));
     if (out_dt == HFB_F32)
         g_launch_err = launch_pdl(latent_split_kernel<float>, grid, block, smem, (cudaStream_t)s, src, splits, q_w, kv_w, eps, cos_sin,
-                                  n_positions, positions, slots, (float *)cq_out, (float *)cache, (long long)cache_slots, T, q_rank, kv_rank, rot, error_word());
+                                  n_positions, positions, slots, (float *)cq_out, (float *)cache, (long long)cache_slots, T, q_rank, kv_rank, rot,
+                                  row_stride, (float *)gate_out, n_gate, error_word());
     else
         g_launch_err = launch_pdl(latent_split_kernel<__nv_bfloat16>, grid, block, smem, (cudaStream_t)s, src, splits, q_w, kv_w, eps, cos_sin,
                                   n_positions, positions, slots, (__nv_bfloat16 *)cq_out, (__nv_bfloat16 *)cache, (long long)cache_slots, T, q_rank,
-                                  kv_rank, rot, error_word());
+                                  kv_rank, rot, row_stride, (__nv_bfloat16 *)gate_out, n_gate, error_word());
     return check_pdl_launch(g_launch_err, "latent_split");
 }
 
@@ -371,7 +409,7 @@ extern "C" int hfb_latent_query_rope(const float *src, int splits, const float *
 }
 
 extern "C" int hfb_headwise_linear(const void *in, int in_dt, const void *w, int w_dt, void *out, int out_dt, int T, int H, int N,
-                                   int K, int in_row, int out_row, hfb_stream s)
+                                   int K, int in_row, int out_row, const void *gate, hfb_stream s)
 {
     if (T <= 0) return HFB_OK;
     if (!valid_dt(in_dt) || !valid_dt(w_dt) || !valid_dt(out_dt) || H <= 0 || N <= 0 || K <= 0 || in_row < K || out_row < N)
@@ -383,12 +421,12 @@ extern "C" int hfb_headwise_linear(const void *in, int in_dt, const void *w, int
         const dim3 mgrid((T + HM_T - 1) / HM_T, headwise_tiles_y(T, N, K), H);
         g_launch_err = launch_pdl(headwise_mma_kernel<0>, mgrid, dim3(128), 0, (cudaStream_t)s, (const __nv_bfloat16 *)in, (const float *)nullptr, 1,
                                   (const __nv_bfloat16 *)w, (__nv_bfloat16 *)out, T, H, N, K, in_row, out_row, (const float *)nullptr, 0,
-                                  (const int32_t *)nullptr, 0, 0, error_word());
+                                  (const int32_t *)nullptr, 0, 0, (const __nv_bfloat16 *)gate, error_word());
         return check_pdl_launch(g_launch_err, "headwise_linear");
     }
     const dim3 grid((T + HW_TT - 1) / HW_TT, (N + HW_NT - 1) / HW_NT, H);
     g_launch_err = launch_pdl(headwise_linear_kernel<float, float, float>, grid, dim3(256), 0, (cudaStream_t)s, (const float *)in, (const float *)w,
-                              (float *)out, T, H, N, K, in_row, out_row);
+                              (float *)out, T, H, N, K, in_row, out_row, (const float *)gate);
     return check_pdl_launch(g_launch_err, "headwise_linear");
 }
 
@@ -403,6 +441,6 @@ extern "C" int hfb_latent_query_absorb(const float *src, int splits, const float
     const dim3 grid((T + HM_T - 1) / HM_T, headwise_tiles_y(T, kv_rank, d), H);
     g_launch_err = launch_pdl(headwise_mma_kernel<1>, grid, dim3(128), 0, (cudaStream_t)s, (const __nv_bfloat16 *)nullptr, src, splits,
                               (const __nv_bfloat16 *)w_ukt, (__nv_bfloat16 *)q_att, T, H, kv_rank, d, d + rot, kv_rank + rot, cos_sin, n_positions,
-                              positions, rot, kv_rank, error_word());
+                              positions, rot, kv_rank, (const __nv_bfloat16 *)nullptr, error_word());
     return check_pdl_launch(g_launch_err, "latent_query_absorb");
 }

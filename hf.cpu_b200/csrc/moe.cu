@@ -25,6 +25,20 @@ __device__ __forceinline__ float moe_act(float v, int act)
     return v;
 }
 
+// The two halves of a gated pair: act(g) * u, or, for HFB_ACT_CLAMPED_GLU, min(g, limit) sigmoid(alpha min(g, limit)) *
+// (clamp(u, -limit, limit) + offset).
+struct GluClamp { float limit, alpha, offset; };
+
+__device__ __forceinline__ float moe_glu(float g, float u, int act, const GluClamp &c)
+{
+    if (act == HFB_ACT_CLAMPED_GLU) {
+        g = fminf(g, c.limit);
+        u = fminf(fmaxf(u, -c.limit), c.limit);
+        return g / (1.0f + expf(-c.alpha * g)) * (u + c.offset);
+    }
+    return moe_act(g, act) * u;
+}
+
 // The choice of experts from the router's logits z [splits, T, E] (float32: partial sums of the router's product,
 // summed in split order, plus its bias; finished logits have one split and no bias): one warp per token; the `top`
 // largest, the lower index among equals; weights = softmax over the chosen logits only.  smem per warp: E logits, `top`
@@ -71,16 +85,17 @@ moe_topk_kernel(const float *zs, int splits, const void *bias, int bias_dt, int 
     }
 }
 
-// A router that scores with a softmax over all of its outputs and chooses among groups: z [splits, T, E] as above;
-// s = softmax(z) over all E; the choice score of an output is s + correction; the E outputs form `n_groups` equal groups
-// of neighbours, a group's score is its largest choice score, and only the outputs of the `keep` best groups can be
-// chosen (the lower group among equals); of those the `top` largest choice scores choose (the lower index among equals).
-// weights = s of the chosen (without the correction) * scale, not renormalised.  An index at or above the number of real
-// experts names an identity expert; whoever reads `ids` decides what that means.  One warp per token; smem per warp:
-// 2 E + n_groups floats.
+// A router that scores every output and chooses among groups: z [splits, T, E] as above; s = softmax(z) over all E, or (SIGMOID)
+// sigmoid(z) each by itself; the choice score of an output is s + correction; the E outputs form `n_groups` equal groups
+// of neighbours, a group's score is the sum of its `group_best` (1 or 2) largest choice scores, and only the outputs of the
+// `keep` best groups can be chosen (the lower group among equals); of those the `top` largest choice scores choose (the
+// lower index among equals).  weights = s of the chosen (without the correction), with `renorm` divided by their sum +
+// 1e-20, times `scale`.  An index at or above the number of real experts names an identity expert; whoever reads `ids`
+// decides what that means.  One warp per token; smem per warp: 2 E + n_groups floats.
+template <bool SIGMOID>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-moe_route_softmax_kernel(const float *zs, int splits, const void *correction, int corr_dt, int T, int E, int top, int n_groups,
-                         int keep, float scale, int32_t *ids, float *weights)
+moe_route_scored_kernel(const float *zs, int splits, const void *correction, int corr_dt, int T, int E, int top, int n_groups,
+                        int keep, int group_best, int renorm, float scale, int32_t *ids, float *weights)
 {
     pdl_entry();
     pdl_sync_small();
@@ -89,20 +104,23 @@ moe_route_softmax_kernel(const float *zs, int splits, const void *correction, in
     const int t = blockIdx.x * ROUTE_WARPS + warp;
     if (t >= T) return;
     float *sc = route_smem + (size_t)warp * (2 * E + n_groups), *ch = sc + E, *gs = ch + E;
+    const size_t plane = (size_t)T * E;
     float m = -INFINITY;
     for (int e = lane; e < E; e += 32) {
-        float v = 0.f;
-        for (int s = 0; s < splits; s++) v += zs[((size_t)s * T + t) * E + e];
+        const float v = plane_sum(zs + (size_t)t * E + e, splits, plane);
         sc[e] = v;
         m = fmaxf(m, v);
     }
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int e = lane; e < E; e += 32) { const float p = expf(sc[e] - m); sc[e] = p; sum += p; }
-    sum = warp_sum(sum);
-    const float inv = 1.0f / sum;
+    float inv = 1.0f;
+    if (!SIGMOID) {
+        m = warp_max(m);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) { const float p = expf(sc[e] - m); sc[e] = p; sum += p; }
+        sum = warp_sum(sum);
+        inv = 1.0f / sum;
+    }
     for (int e = lane; e < E; e += 32) {
-        const float p = sc[e] * inv;
+        const float p = SIGMOID ? 1.0f / (1.0f + expf(-sc[e])) : sc[e] * inv;
         sc[e] = p;
         ch[e] = correction ? p + load_any(correction, corr_dt, e) : p;
     }
@@ -110,9 +128,13 @@ moe_route_softmax_kernel(const float *zs, int splits, const void *correction, in
     if (n_groups > 1 && keep < n_groups) {
         const int per = E / n_groups;
         for (int g = lane; g < n_groups; g += 32) {
-            float b = -INFINITY;
-            for (int i = 0; i < per; i++) b = fmaxf(b, ch[g * per + i]);
-            gs[g] = b;
+            float b = -INFINITY, b2 = -INFINITY;           // the largest and the second largest
+            for (int i = 0; i < per; i++) {
+                const float v = ch[g * per + i];
+                b2 = fmaxf(b2, fminf(b, v));
+                b = fmaxf(b, v);
+            }
+            gs[g] = group_best > 1 && per > 1 ? b + b2 : b;
         }
         __syncwarp();
         // a group is kept when fewer than `keep` groups come before it in the order (score descending, index ascending)
@@ -125,6 +147,7 @@ moe_route_softmax_kernel(const float *zs, int splits, const void *correction, in
         }
         __syncwarp();
     }
+    float total = 0.f;                                     // of the chosen scores, in the order of the choice
     for (int j = 0; j < top; j++) {
         float best = -INFINITY;
         int bi = 0x7fffffff;
@@ -139,12 +162,18 @@ moe_route_softmax_kernel(const float *zs, int splits, const void *correction, in
             if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
         }
         if (bi == 0x7fffffff) bi = 0;                 // (nothing left to choose from)
+        const float w = sc[bi];
+        total += w;
         if (lane == 0) {
             ids[(size_t)t * top + j] = bi;
-            weights[(size_t)t * top + j] = sc[bi] * scale;
+            weights[(size_t)t * top + j] = w * scale;
             ch[bi] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (renorm) {
+        const float f = 1.0f / (total + 1e-20f);
+        for (int j = lane; j < top; j += 32) weights[(size_t)t * top + j] *= f;
     }
 }
 
@@ -189,7 +218,7 @@ constexpr int GT = 64, GK = 16;       // tile of 64 places x 64 features, 16 of 
 
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(256)
-moe_gemm_kernel(const TA *__restrict__ a, const TW *__restrict__ w, void *out, int out_dt, int act, int N, int K,
+moe_gemm_kernel(const TA *__restrict__ a, const TW *__restrict__ w, void *out, int out_dt, int act, GluClamp clamp, int N, int K,
                 const int32_t *order, int src_div, int scatter, const int32_t *tile_expert, const int32_t *tile_p0,
                 const int32_t *tile_n, const int32_t *n_tiles)
 {
@@ -259,7 +288,7 @@ moe_gemm_kernel(const TA *__restrict__ a, const TW *__restrict__ w, void *out, i
             const int gn = n0 + tx * 4 + j;
             if (gn >= N) continue;
             if (glu) {              // rows of w alternate gate, up: features (2f, 2f + 1) give out[f] = act(gate) * up
-                if (!(j & 1)) store_any(out, out_dt, (size_t)dst * (N / 2) + gn / 2, moe_act(acc[i][j], act) * acc[i][j + 1]);
+                if (!(j & 1)) store_any(out, out_dt, (size_t)dst * (N / 2) + gn / 2, moe_glu(acc[i][j], acc[i][j + 1], act, clamp));
                 continue;
             }
             store_any(out, out_dt, (size_t)dst * N + gn, moe_act(acc[i][j], act));
@@ -306,7 +335,7 @@ constexpr size_t MMA_SMEM = (size_t)MSTAGES * (MT + MN) * (MK + MPAD) * sizeof(_
 
 __global__ void __launch_bounds__(256)
 moe_gemm_mma_kernel(const __nv_bfloat16 *__restrict__ a, const __nv_bfloat16 *__restrict__ w, void *out, int out_dt, int act,
-                    int N, int K, const int32_t *order, int src_div, int scatter, const int32_t *tile_expert,
+                    GluClamp clamp, int N, int K, const int32_t *order, int src_div, int scatter, const int32_t *tile_expert,
                     const int32_t *tile_p0, const int32_t *tile_n, const int32_t *n_tiles)
 {
     const int glu = act >> 8;          // HFB_ACT_GLU set: see the epilogue
@@ -412,7 +441,7 @@ moe_gemm_mma_kernel(const __nv_bfloat16 *__restrict__ a, const __nv_bfloat16 *__
                     const int gn = n0 + 64 * wn + nt * 8 + 2 * t + j;
                     if (gn >= n_end) continue;
                     if (glu) {
-                        if (j == 0) store_any(out, out_dt, (size_t)dst * (N / 2) + gn / 2, moe_act(acc[m][nt][2 * half], act) * acc[m][nt][2 * half + 1]);
+                        if (j == 0) store_any(out, out_dt, (size_t)dst * (N / 2) + gn / 2, moe_glu(acc[m][nt][2 * half], acc[m][nt][2 * half + 1], act, clamp));
                         continue;
                     }
                     store_any(out, out_dt, (size_t)dst * N + gn, moe_act(acc[m][nt][2 * half + j], act));
@@ -431,7 +460,7 @@ constexpr size_t SMALL_SMEM = (size_t)ST_STAGES * (ST_ROWS + ST_N) * (ST_K + MPA
 
 __global__ void __launch_bounds__(128)
 moe_gemm_small_kernel(const __nv_bfloat16 *__restrict__ a, const __nv_bfloat16 *__restrict__ w, void *out, int out_dt, int act,
-                      int N, int K, const int32_t *order, int src_div, int scatter, const int32_t *tile_expert,
+                      GluClamp clamp, int N, int K, const int32_t *order, int src_div, int scatter, const int32_t *tile_expert,
                       const int32_t *tile_p0, const int32_t *tile_n, const int32_t *n_tiles)
 {
     const int glu = act >> 8;          // HFB_ACT_GLU set: see the epilogue
@@ -516,7 +545,7 @@ moe_gemm_small_kernel(const __nv_bfloat16 *__restrict__ a, const __nv_bfloat16 *
                 const int gn = n0 + 16 * warp + nt * 8 + 2 * t + j;
                 if (gn >= N) continue;
                 if (glu) {
-                    if (j == 0) store_any(out, out_dt, (size_t)dst * (N / 2) + gn / 2, moe_act(acc[nt][2 * half], act) * acc[nt][2 * half + 1]);
+                    if (j == 0) store_any(out, out_dt, (size_t)dst * (N / 2) + gn / 2, moe_glu(acc[nt][2 * half], acc[nt][2 * half + 1], act, clamp));
                     continue;
                 }
                 store_any(out, out_dt, (size_t)dst * N + gn, moe_act(acc[nt][2 * half + j], act));
@@ -562,18 +591,24 @@ extern "C" int hfb_moe_topk(const float *z, int splits, const void *bias, int bi
     return check_pdl_launch(g_launch_err, "moe_topk");
 }
 
-extern "C" int hfb_moe_route_softmax(const float *z, int splits, const void *correction, int corr_dt, int T, int E, int top,
-                                     int n_groups, int keep, float scale, int32_t *ids, float *weights, hfb_stream s)
+extern "C" int hfb_moe_route_scored(const float *z, int splits, const void *correction, int corr_dt, int T, int E, int top, int score,
+                                    int n_groups, int keep, int group_best, int renorm, float scale, int32_t *ids, float *weights,
+                                    hfb_stream s)
 {
     if (T <= 0) return HFB_OK;
     if (E <= 0 || top <= 0 || top > E || splits < 1 || (correction && !valid_dt(corr_dt)) || n_groups < 1 || E % n_groups ||
-        keep < 1 || keep > n_groups || keep * (E / n_groups) < top)
-        return fail(HFB_EINVAL, "moe_route_softmax: bad arguments (outputs=%d top=%d groups=%d keep=%d)", E, top, n_groups, keep);
+        keep < 1 || keep > n_groups || keep * (E / n_groups) < top || score < 0 || score > 1 || group_best < 1 || group_best > 2)
+        return fail(HFB_EINVAL, "moe_route_scored: bad arguments (outputs=%d top=%d groups=%d keep=%d)", E, top, n_groups, keep);
     const size_t smem = (size_t)ROUTE_WARPS * (2 * E + n_groups) * sizeof(float);
-    if (smem > 48 * 1024) return fail(HFB_ENOTSUP, "moe_route_softmax: %d router outputs are more than the kernel takes", E);
-    g_launch_err = launch_pdl(moe_route_softmax_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), smem, (cudaStream_t)s,
-                              z, splits, correction, corr_dt, T, E, top, n_groups, keep, scale, ids, weights);
-    return check_pdl_launch(g_launch_err, "moe_route_softmax");
+    if (smem > 48 * 1024) return fail(HFB_ENOTSUP, "moe_route_scored: %d router outputs are more than the kernel takes", E);
+    const dim3 grid((T + ROUTE_WARPS - 1) / ROUTE_WARPS), block(ROUTE_WARPS * 32);
+    if (score == 1)
+        g_launch_err = launch_pdl(moe_route_scored_kernel<true>, grid, block, smem, (cudaStream_t)s, z, splits, correction, corr_dt, T, E, top, n_groups,
+                                  keep, group_best, renorm, scale, ids, weights);
+    else
+        g_launch_err = launch_pdl(moe_route_scored_kernel<false>, grid, block, smem, (cudaStream_t)s, z, splits, correction, corr_dt, T, E, top, n_groups,
+                                  keep, group_best, renorm, scale, ids, weights);
+    return check_pdl_launch(g_launch_err, "moe_route_scored");
 }
 
 extern "C" int hfb_moe_max_tiles(int pairs, int E, int tile)
@@ -593,16 +628,18 @@ extern "C" int hfb_moe_sort(const int32_t *ids, int pairs, int E, int tile, int3
     return check_pdl_launch(g_launch_err, "moe_sort");
 }
 
-extern "C" int hfb_moe_gemm(const void *a, int a_dt, const void *w, int w_dt, void *out, int out_dt, int act, int N, int K,
+extern "C" int hfb_moe_gemm(const void *a, int a_dt, const void *w, int w_dt, void *out, int out_dt, int act, float limit, float alpha,
+                            float offset, int N, int K,
                             const int32_t *order, int src_div, int scatter, const int32_t *tile_expert, const int32_t *tile_p0,
                             const int32_t *tile_n, const int32_t *n_tiles, int max_tiles, int tile, hfb_stream s)
 {
     if (max_tiles <= 0) return HFB_OK;
-    if (!valid_dt(a_dt) || !valid_dt(w_dt) || !valid_dt(out_dt) || N <= 0 || K <= 0 || tile < 1 || tile > MT || act < 0 || (act & 255) > HFB_ACT_NONE ||
-        (act >> 8) > 1 || ((act >> 8) && (N & 1)))
+    if (!valid_dt(a_dt) || !valid_dt(w_dt) || !valid_dt(out_dt) || N <= 0 || K <= 0 || tile < 1 || tile > MT || act < 0 ||
+        ((act & 255) > HFB_ACT_NONE && act != (HFB_ACT_GLU | HFB_ACT_CLAMPED_GLU)) || (act >> 8) > 1 || ((act >> 8) && (N & 1)))
         return fail(HFB_EINVAL, "moe_gemm: bad arguments (N=%d K=%d tile=%d)", N, K, tile);
     if (max_tiles > 65535) return fail(HFB_ENOTSUP, "moe_gemm: %d tiles exceed the grid", max_tiles);
     const dim3 grid((N + GT - 1) / GT, max_tiles);
+    const GluClamp clamp{limit, alpha, offset};
     cudaStream_t st = (cudaStream_t)s;
     if (a_dt == HFB_BF16 && w_dt == HFB_BF16 && (K & 7) == 0 && ((uintptr_t)a & 15) == 0 && ((uintptr_t)w & 15) == 0 &&
         !plain_products()) {
@@ -616,14 +653,14 @@ extern "C" int hfb_moe_gemm(const void *a, int a_dt, const void *w, int w_dt, vo
         }
         if (tile <= ST_ROWS) {                  // tiles of at most 16 places: the form for steps of a few tokens
             g_launch_err = launch_pdl(moe_gemm_small_kernel, dim3((N + ST_N - 1) / ST_N, max_tiles), dim3(128), SMALL_SMEM, st, (const __nv_bfloat16 *)a,
-                                      (const __nv_bfloat16 *)w, out, out_dt, act, N, K, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles);
+                                      (const __nv_bfloat16 *)w, out, out_dt, act, clamp, N, K, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles);
             return check_pdl_launch(g_launch_err, "moe_gemm_small");
         }
-        g_launch_err = launch_pdl(moe_gemm_mma_kernel, dim3((N + MN - 1) / MN, max_tiles), dim3(256), MMA_SMEM, st, (const __nv_bfloat16 *)a, (const __nv_bfloat16 *)w, out, out_dt, act, N, K,
+        g_launch_err = launch_pdl(moe_gemm_mma_kernel, dim3((N + MN - 1) / MN, max_tiles), dim3(256), MMA_SMEM, st, (const __nv_bfloat16 *)a, (const __nv_bfloat16 *)w, out, out_dt, act, clamp, N, K,
                                   order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles);
         return check_pdl_launch(g_launch_err, "moe_gemm_mma");
     }
-#define LAUNCH(TA, TW) g_launch_err = launch_pdl(moe_gemm_kernel<TA, TW>, dim3(grid.x, grid.y, (tile + GT - 1) / GT), dim3(256), 0, st, (const TA *)a, (const TW *)w, out, out_dt, act, N, K, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles)
+#define LAUNCH(TA, TW) g_launch_err = launch_pdl(moe_gemm_kernel<TA, TW>, dim3(grid.x, grid.y, (tile + GT - 1) / GT), dim3(256), 0, st, (const TA *)a, (const TW *)w, out, out_dt, act, clamp, N, K, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles)
     if (a_dt == HFB_F32 && w_dt == HFB_F32) LAUNCH(float, float);
     else if (a_dt == HFB_F32) LAUNCH(float, __nv_bfloat16);
     else if (w_dt == HFB_F32) LAUNCH(__nv_bfloat16, float);

@@ -51,6 +51,8 @@ def step_flops(model, q_lens: Sequence[int], kv_lens: Sequence[int], logit_rows:
     for e in model.plan.schedule:
         layer = model.layers[e.layer]
         total += layer.mixer.flops(q_lens, kv_lens) + (layer.ffn.flops(sum(q_lens)) if layer.ffn is not None else 0.0)
+        if e.enter is not None:
+            total += model.transitions[e.enter[0]].flops(sum(q_lens))
     return total + model.head.flops(logit_rows)
 
 

@@ -27,7 +27,7 @@ class PhaseProfile:
     ``kernels.phase(name)``; while the profile is on, each phase is bracketed by CUDA events on the current stream
     and ``take()`` returns milliseconds per name and clears them.  Off, ``phase`` costs one attribute test.  The
     reference keeps per-phase accumulators with the same names (src/model.h:75-79, src/ops.c:593-604)."""
-    NAMES = ("embed", "glue", "qkv", "attn", "wo", "gate_up", "silu", "down", "head", "quant", "sample")
+    NAMES = ("embed", "glue", "qkv", "attn", "wo", "gate_up", "silu", "down", "join", "head", "quant", "sample")
 
     class _Null:
         def __enter__(self):
@@ -372,6 +372,36 @@ def linear_dyt_residual(a, w, bias, y_buf, post, residual, nxt=None, out=None, m
         backend().linear_dyt_residual(a, w, bias, y_buf, post, residual, nxt, out, mix=mix)
 
 
+def rms_tail(y, splits: int, residual, post=None, nxt=None, out=None, bias=None, mix=None, base=None) -> None:
+    """What ends a sublayer (or a step between layers) in one pass over the float32 stream:
+
+        v = sum of the ``splits`` planes of y (+ ``bias``) (+ the weighted rows of ``mix``)
+        v = v / sqrt(mean(v^2) + eps) * w          with ``post`` = (w, eps)
+        residual = (``base``, else residual) + v
+        out = residual / sqrt(mean(residual^2) + eps) * w with ``nxt`` = (w, eps), or residual as it is with ``nxt`` = "copy"
+
+    y float32 [splits, M, N], or None (then only mix, or nothing but ``out``); ``mix`` = (rows float32 [M * top, N], weights
+    float32 [M, top]), summed in the order of the rows."""
+    M, N = residual.shape
+    some = y is not None or mix is not None
+    _need(residual.dtype == torch.float32, "rms_tail: the stream is float32")
+    _need(y is None or (y.dtype == torch.float32 and splits >= 1 and y.numel() >= splits * M * N), "rms_tail: y is float32 [splits, M, N]")
+    _mix_ok(mix, residual, "rms_tail")
+    _need(post is None or (post[0].shape == (N,) and some), "rms_tail: the norm of nothing")
+    _need(bias is None or (bias.shape == (N,) and some), "rms_tail: the bias is [N] and comes with a sum")
+    _need(base is None or (base.shape == residual.shape and base.dtype == torch.float32 and some), "rms_tail: the base is float32 like the stream")
+    _need((nxt is None) == (out is None), "rms_tail: what follows and its output come together")
+    _need(nxt is None or (out.shape == residual.shape and (nxt == "copy" or nxt[0].shape == (N,))), "rms_tail: output shape mismatch")
+    backend().rms_tail(y, int(splits) if y is not None else 0, residual, post, nxt, out, bias=bias, mix=mix, base=base)
+
+
+def linear_rms_tail(a, w, y_buf, residual, bias=None, post=None, nxt=None, out=None, mix=None, base=None) -> None:
+    """:func:`rms_tail` behind the product ``a @ w.T``: the pass sums the product's partial sums where it is split over its
+    inner dimension, else the product is stored in ``y_buf`` ([M, N] float32) first."""
+    y, splits = product_sums(a, w, y_buf)
+    rms_tail(y, splits, residual, post=post, nxt=nxt, out=out, bias=bias, mix=mix, base=base)
+
+
 def linear_rope_norm_kv(a, w, bias, qkv_buf, cos_sin, n_rot, positions, slots, q_out, k_cache, v_cache, H, G, d, dv,
                         norm_eps, norm_weights=None, value_mix=None, pairing: str = "half") -> None:
     """The q|k|v product and its tail for attention with unit-rms queries and keys: row = [H heads of d | G key heads
@@ -412,13 +442,19 @@ def linear_rope_norm_kv(a, w, bias, qkv_buf, cos_sin, n_rot, positions, slots, q
                                   H, G, d, dv, None if norm_eps is None else float(norm_eps), **extra)
 
 
-def linear_latent_split(a, w, buf, q_norm_w, kv_norm_w, eps, cos_sin, positions, slots, cq_out, cache, q_rank, kv_rank, rot) -> None:
+def linear_latent_split(a, w, buf, q_norm_w, kv_norm_w, eps, cos_sin, positions, slots, cq_out, cache, q_rank, kv_rank, rot,
+                        gate_out=None) -> None:
     """Latent attention's down product and its tail: row = a @ w.T = [q_rank | kv_rank | rot]; the first two parts are
     normed (x / sqrt(mean(x^2) + eps) times a float32 weight), the query latent goes to ``cq_out``, the key/value latent
     and the last part, rotated in pairs (2i, 2i + 1), form the token's row of ``cache`` [pages, block, 1, kv_rank + rot].
-    ``buf`` [T, row] float32 is scratch."""
-    C = q_rank + kv_rank + rot
-    _need(w.shape[0] == C and a.shape[1] == w.shape[1] and buf.shape == (a.shape[0], C) and buf.dtype == torch.float32,
+    ``gate_out`` ([T, gates] in the run's type): the row ends in that many more columns, whose sigmoid goes there; the row
+    may have padding behind it.  ``buf`` [T, row] float32 is scratch."""
+    n_gate = 0 if gate_out is None else gate_out.shape[1]
+    C = w.shape[0]
+    _need(C == q_rank + kv_rank + rot if gate_out is None else
+          (C >= q_rank + kv_rank + rot + n_gate and gate_out.shape[0] == a.shape[0] and gate_out.dtype == cq_out.dtype),
+          "linear_latent_split: row or gate mismatch")
+    _need(a.shape[1] == w.shape[1] and buf.shape == (a.shape[0], C) and buf.dtype == torch.float32,
           "linear_latent_split: shape mismatch")
     _need(q_norm_w.shape == (q_rank,) and kv_norm_w.shape == (kv_rank,) and q_norm_w.dtype == kv_norm_w.dtype == torch.float32,
           "linear_latent_split: norm weights are float32 [q_rank] and [kv_rank]")
@@ -427,7 +463,7 @@ def linear_latent_split(a, w, buf, q_norm_w, kv_norm_w, eps, cos_sin, positions,
     _need(rot % 2 == 0 and (rot == 0 or (cos_sin is not None and cos_sin.shape[1:] == (rot // 2, 2) and cos_sin.dtype == torch.float32)),
           "linear_latent_split: cos/sin table must be float32 [positions, rot/2, 2]")
     backend().linear_latent_split(a, w, buf, q_norm_w, kv_norm_w, float(eps), cos_sin, positions, slots, cq_out, cache,
-                                  int(q_rank), int(kv_rank), int(rot))
+                                  int(q_rank), int(kv_rank), int(rot), **({"gate_out": gate_out} if gate_out is not None else {}))
 
 
 def linear_latent_query(a, w, buf, cos_sin, positions, q_plain, q_att, H, d, rot, att_col) -> None:
@@ -464,13 +500,15 @@ def linear_latent_query_absorb(a, w_uq, buf, cos_sin, positions, w_ukt, q_plain,
     headwise_linear(q_plain, w_ukt, q_att, H, d, R + rot)
 
 
-def headwise_linear(x, w, out, H: int, in_row: int, out_row: int) -> None:
+def headwise_linear(x, w, out, H: int, in_row: int, out_row: int, gate=None) -> None:
     """A product per head: out[t, h, :N] = w[h] @ x[t, h, :K] with w [H, N, K]; a row of ``x`` holds H heads ``in_row``
-    apart, a row of ``out`` H heads ``out_row`` apart (a head's result may be the first N columns of a wider row)."""
+    apart, a row of ``out`` H heads ``out_row`` apart (a head's result may be the first N columns of a wider row).
+    ``gate`` ([T, H * N] in the run's type): factors on the result."""
     _need(w.dim() == 3 and w.shape[0] == H and x.shape[1] == H * in_row and out.shape == (x.shape[0], H * out_row)
           and in_row >= w.shape[2] and out_row >= w.shape[1], "headwise_linear: shape mismatch")
     _need(x.dtype == out.dtype == w.dtype, "headwise_linear: element types differ")
-    backend().headwise_linear(x, w, out, int(H), int(in_row), int(out_row))
+    _need(gate is None or (gate.shape == (x.shape[0], H * w.shape[1]) and gate.dtype == out.dtype), "headwise_linear: gate is [T, H * N]")
+    backend().headwise_linear(x, w, out, int(H), int(in_row), int(out_row), **({"gate": gate} if gate is not None else {}))
 
 
 def linear_glu(a: torch.Tensor, w: torch.Tensor, gu_buf: torch.Tensor, out: torch.Tensor, act: str, bias=None, clamp=None) -> None:
@@ -536,14 +574,18 @@ def moe_group(ids, experts: int, order, tile_expert, tile_p0, tile_n, n_tiles) -
 
 
 def moe_gemm(a, w, out, act: str, order, src_div: int, scatter: bool, tile_expert, tile_p0, tile_n, n_tiles, pairs: int,
-             glu: bool = False) -> None:
+             glu: bool = False, clamp=None) -> None:
     """Grouped product over the places of :func:`moe_group`: out[dst(p)] = act(a[src(p)] @ w[expert(p)].T) with
     w [E, N, K]; src(p) = order[p] // src_div if src_div else p; dst(p) = order[p] if scatter else p.  ``glu``: the rows
-    of an expert's matrix alternate gate, up, and out [.., N / 2] = act(gate) * up."""
+    of an expert's matrix alternate gate, up, and out [.., N / 2] = act(gate) * up; act "clamped" with ``clamp`` = (limit,
+    alpha, offset) as in :func:`linear_glu`."""
     _need(w.dim() == 3 and a.shape[1] == w.shape[2], "moe_gemm: shape mismatch")
+    _need((act == "clamped") == (clamp is not None) and (clamp is None or glu), "moe_gemm: the clamped form is gated and comes with its constants")
     _need(out.shape[1] == (w.shape[1] // 2 if glu else w.shape[1]) and (not glu or w.shape[1] % 2 == 0), "moe_gemm: output width mismatch")
-    backend().moe_gemm(a, w, out, _act(act) | (ACT_GLU if glu else 0), order, int(src_div), bool(scatter), tile_expert, tile_p0,
-                       tile_n, n_tiles, moe_max_tiles(int(pairs), w.shape[0]), moe_tile(int(pairs)))
+    code = (ACT_CLAMPED_GLU if act == "clamped" else _act(act)) | (ACT_GLU if glu else 0)
+    backend().moe_gemm(a, w, out, code, order, int(src_div), bool(scatter), tile_expert, tile_p0,
+                       tile_n, n_tiles, moe_max_tiles(int(pairs), w.shape[0]), moe_tile(int(pairs)),
+                       **({"clamp": tuple(float(x) for x in clamp)} if clamp is not None else {}))
 
 
 def moe_combine(y, weights, out) -> None:
@@ -553,19 +595,26 @@ def moe_combine(y, weights, out) -> None:
     backend().moe_combine(y, weights, out)
 
 
-def moe_route_softmax(h, w, correction, top: int, n_groups: int, keep: int, scale: float, ids, weights, logits) -> None:
-    """Router whose scores are a softmax over all of its outputs: s = softmax(h @ w.T) (float32); choice score = s +
-    ``correction`` (or s); the outputs form ``n_groups`` equal groups of neighbours, a group's score is its largest
-    choice score, and only outputs of the ``keep`` best groups can be chosen; ``ids`` = the ``top`` largest choice scores
-    (largest first, the lower index among equals), ``weights`` = s[ids] * scale, not renormalised."""
+ROUTE_SCORES = {"softmax": 0, "sigmoid": 1}
+
+
+def moe_route_scored(h, w, correction, top: int, ids, weights, logits, score: str = "softmax", n_groups: int = 1, keep: int = 1,
+                     group_best: int = 1, renorm: bool = False, scale: float = 1.0) -> None:
+    """Router that scores every output and may choose among groups: s = softmax(z) over all outputs or sigmoid(z), z = h @
+    w.T (float32); choice score = s + ``correction`` (or s); the outputs form ``n_groups`` equal groups of neighbours, a
+    group's score is the sum of its ``group_best`` (1 or 2) largest choice scores (of the one it has, if it has one only),
+    and only outputs of the ``keep`` best groups can be chosen; ``ids`` = the ``top`` largest choice scores (largest first, the
+    lower index among equals), ``weights`` = s[ids], with ``renorm`` divided by their sum + 1e-20, times ``scale``."""
     T, E = h.shape[0], w.shape[0]
-    _need(h.shape[1] == w.shape[1] and (correction is None or correction.shape == (E,)) and 1 <= top <= E, "moe_route_softmax: shape mismatch")
+    _need(h.shape[1] == w.shape[1] and (correction is None or correction.shape == (E,)) and 1 <= top <= E, "moe_route_scored: shape mismatch")
     _need(n_groups >= 1 and E % n_groups == 0 and 1 <= keep <= n_groups and keep * (E // n_groups) >= top,
-          "moe_route_softmax: the kept groups must hold at least `top` outputs")
+          "moe_route_scored: the kept groups must hold at least `top` outputs")
+    _need(score in ROUTE_SCORES and group_best in (1, 2), "moe_route_scored: score softmax or sigmoid, a group's best one or two")
     _need(ids.shape == (T, top) and ids.dtype == torch.int32 and weights.shape == (T, top) and weights.dtype == torch.float32,
-          "moe_route_softmax: ids int32 [T, top], weights float32 [T, top]")
-    _need(logits.shape == (T, E) and logits.dtype == torch.float32, "moe_route_softmax: logits float32 [T, outputs]")
-    backend().moe_route_softmax(h, w, correction, int(top), int(n_groups), int(keep), float(scale), ids, weights, logits)
+          "moe_route_scored: ids int32 [T, top], weights float32 [T, top]")
+    _need(logits.shape == (T, E) and logits.dtype == torch.float32, "moe_route_scored: logits float32 [T, outputs]")
+    backend().moe_route_scored(h, w, correction, int(top), ids, weights, logits, ROUTE_SCORES[score], int(n_groups), int(keep),
+                               int(group_best), bool(renorm), float(scale))
 
 
 def product_sums(a, w, buf, finished: bool = False):
@@ -732,15 +781,18 @@ def _decay_ok(q, k, u, H, Hq, d, dv, what):
     _need(dp <= SCAN_MAX_HEAD, f"{what}: key heads above {SCAN_MAX_HEAD} are not supported")
 
 
-def rotate_heads(src, splits: int, row: int, cos_sin, n_rot: int, positions, k_scale: float, q, k, u, H: int, d: int, dv: int) -> None:
-    """Operands of retention from the sums of its product (``splits`` float32 planes [T, row]: H query heads of d, H key
-    heads of d, H value heads of dv, ...): rotation of the first ``n_rot`` dimensions (i with i + n_rot/2) of queries and
+def rotate_heads(src, splits: int, row: int, cos_sin, n_rot: int, positions, k_scale: float, q, k, u, H: int, d: int, dv: int,
+                 activation=None) -> None:
+    """Operands of a recurrence with a fixed decay from the sums of its product (``splits`` float32 planes [T, row]: H query
+    heads of d, H key heads of d, H value heads of dv, ...): ``activation`` ("silu" or None) of all three, rotation of the first ``n_rot`` dimensions (i with i + n_rot/2) of queries and
     keys, keys times ``k_scale``; q, k, u as :func:`decay_scan` takes them."""
     _decay_ok(q, k, u, H, H, d, dv, "rotate_heads")
     _need(src.dtype == torch.float32 and src.numel() >= splits * q.shape[0] * row and row >= H * (2 * d + dv), "rotate_heads: rows are float32 [splits, T, row]")
     _need(n_rot % 2 == 0 and 0 <= n_rot <= d and (n_rot == 0 or (cos_sin is not None and cos_sin.shape[1:] == (n_rot // 2, 2)
           and cos_sin.dtype == torch.float32)), "rotate_heads: cos/sin table must be float32 [positions, n_rot/2, 2]")
-    backend().rotate_heads(src, int(splits), int(row), cos_sin, int(n_rot), positions, float(k_scale), q, k, u, int(H), int(d), int(dv))
+    _need(activation in (None, "silu"), "rotate_heads: the activation is silu or none")
+    backend().rotate_heads(src, int(splits), int(row), cos_sin, int(n_rot), positions, float(k_scale), q, k, u, int(H), int(d), int(dv),
+                           **({"silu": True} if activation else {}))
 
 
 def state_space_operands(src, splits: int, row: int, conv_w, conv_b, dt_bias, rate, carried, ctx, q, k, u, step, la, H: int, G: int,
@@ -779,15 +831,18 @@ def decay_scan(q, k, u, la, step, skip, state, ctx, o, H: int, Hq: int, d: int, 
     backend().decay_scan(q, k, u, la, step, skip, state, ctx, o, int(H), int(Hq), int(d), int(dv), chunks or {})
 
 
-def part_norm_gate(o, parts: int, eps: float, g, g_splits: int, g_stride: int, g_col0: int, w, gate_first: bool, out) -> None:
+def part_norm_gate(o, parts: int, eps: float, g, g_splits: int, g_stride: int, g_col0: int, w, gate_first: bool, out,
+                   gate: str = "silu") -> None:
     """out = the rows of o (float32 [T, C]) in ``parts`` equal parts, each divided by its own root mean square, times ``w``
-    (float32 [C]) where given; silu(g) multiplies before the norm (``gate_first``) or after it, g the sum of ``g_splits``
+    (float32 [C]) where given; silu(g) (or sigmoid(g): ``gate``) multiplies before the norm (``gate_first``) or after it, g the sum of ``g_splits``
     float32 planes [T, g_stride] read from column ``g_col0`` on.  ``out`` may be a column slice of a wider array."""
     T, C = o.shape
     _need(o.dtype == torch.float32 and out.shape == (T, C) and out.stride(1) == 1 and C % parts == 0, "part_norm_gate: shape mismatch")
     _need(g.dtype == torch.float32 and g.numel() >= g_splits * T * g_stride and g_col0 + C <= g_stride, "part_norm_gate: g is float32 [splits, T, stride]")
     _need(w is None or (w.shape == (C,) and w.dtype == torch.float32), "part_norm_gate: the weight is float32 [C]")
-    backend().part_norm_gate(o, int(parts), float(eps), g, int(g_splits), int(g_stride), int(g_col0), w, bool(gate_first), out)
+    _need(gate in ("silu", "sigmoid"), "part_norm_gate: gate is 'silu' or 'sigmoid'")
+    backend().part_norm_gate(o, int(parts), float(eps), g, int(g_splits), int(g_stride), int(g_col0), w, bool(gate_first), out,
+                             **({"gate": gate} if gate != "silu" else {}))
 
 
 # ---- attention normed over the whole projection, head gates -------------------------------------------------------

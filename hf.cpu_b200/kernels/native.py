@@ -427,6 +427,18 @@ class NativeBackend:
             _p(n[2]), c_int(_dt(n[1]) if nxt else 0), _p(out), c_int(_dt(out) if out is not None else 0), c_int(M), c_int(E),
             self._stream()), "dyt_residual")
 
+    def rms_tail(self, y, splits, residual, post, nxt, out, bias=None, mix=None, base=None):
+        post_w, post_eps = post or (None, 0.0)
+        nxt_w, nxt_eps = nxt if isinstance(nxt, tuple) else (None, 0.0)
+        mix_y, mix_w = mix or (None, None)
+        self._on_gpu(y, residual, post_w, nxt_w, out, bias, mix_y, mix_w, base)
+        M, E = residual.shape
+        dt = lambda t: c_int(_dt(t) if t is not None else 0)
+        self._check(self.lib.hfb_rms_tail(
+            _p(y), c_int(splits), _p(bias), dt(bias), _p(mix_y), _p(mix_w), c_int(mix_w.shape[1] if mix_w is not None else 0), _p(post_w),
+            dt(post_w), c_float(post_eps), _p(base), _p(residual), _p(nxt_w), dt(nxt_w), c_float(nxt_eps), _p(out), dt(out), c_int(M), c_int(E),
+            self._stream()), "rms_tail")
+
     def linear_rope_norm_kv(self, a, w, bias, qkv_buf, cos_sin, n_rot, positions, slots, q_out, k_cache, v_cache, H, G, d, dv,
                             norm_eps, norm_weights=None, value_mix=None, pairing="half"):
         self._on_gpu(a, w, bias, cos_sin, positions, slots, q_out, k_cache, v_cache)
@@ -463,14 +475,15 @@ class NativeBackend:
         self.linear(a, w, None, buf, False)
         return buf, 1
 
-    def linear_latent_split(self, a, w, buf, q_norm_w, kv_norm_w, eps, cos_sin, positions, slots, cq_out, cache, q_rank, kv_rank, rot):
-        self._on_gpu(a, w, buf, q_norm_w, kv_norm_w, cos_sin, positions, slots, cq_out, cache)
+    def linear_latent_split(self, a, w, buf, q_norm_w, kv_norm_w, eps, cos_sin, positions, slots, cq_out, cache, q_rank, kv_rank, rot,
+                            gate_out=None):
+        self._on_gpu(a, w, buf, q_norm_w, kv_norm_w, cos_sin, positions, slots, cq_out, cache, gate_out)
         src, splits = self._product_sums(a, w, buf)
         self._check(self.lib.hfb_latent_split(
             _p(src), c_int(splits), _p(q_norm_w), _p(kv_norm_w), c_float(eps), _p(cos_sin),
             c_int(cos_sin.shape[0] if cos_sin is not None else 0), _p(positions), _p(slots), _p(cq_out), _p(cache), c_int(_dt(cq_out)),
-            c_int64(cache.shape[0] * cache.shape[1]), c_int(a.shape[0]), c_int(q_rank), c_int(kv_rank), c_int(rot), self._stream()),
-            "latent_split")
+            c_int64(cache.shape[0] * cache.shape[1]), c_int(a.shape[0]), c_int(q_rank), c_int(kv_rank), c_int(rot), c_int(w.shape[0]),
+            _p(gate_out), c_int(gate_out.shape[1] if gate_out is not None else 0), self._stream()), "latent_split")
 
     def linear_latent_query(self, a, w, buf, cos_sin, positions, q_plain, q_att, H, d, rot, att_col):
         self._on_gpu(a, w, buf, cos_sin, positions, q_plain, q_att)
@@ -487,10 +500,10 @@ class NativeBackend:
             _p(src), c_int(splits), _p(cos_sin), c_int(cos_sin.shape[0] if cos_sin is not None else 0), _p(positions), _p(w_ukt),
             _p(q_att), c_int(a.shape[0]), c_int(H), c_int(d), c_int(rot), c_int(w_ukt.shape[1]), self._stream()), "latent_query_absorb")
 
-    def headwise_linear(self, x, w, out, H, in_row, out_row):
-        self._on_gpu(x, w, out)
+    def headwise_linear(self, x, w, out, H, in_row, out_row, gate=None):
+        self._on_gpu(x, w, out, gate)
         self._check(self.lib.hfb_headwise_linear(_p(x), c_int(_dt(x)), _p(w), c_int(_dt(w)), _p(out), c_int(_dt(out)), c_int(x.shape[0]),
-                                                 c_int(H), c_int(w.shape[1]), c_int(w.shape[2]), c_int(in_row), c_int(out_row),
+                                                 c_int(H), c_int(w.shape[1]), c_int(w.shape[2]), c_int(in_row), c_int(out_row), _p(gate),
                                                  self._stream()), "headwise_linear")
 
     def linear_glu(self, a, w, gu_buf, out, act, bias=None, clamp=None):
@@ -539,13 +552,14 @@ class NativeBackend:
         self._check(self.lib.hfb_moe_topk(_p(src), c_int(splits), _p(b), c_int(_dt(b) if b is not None else 0), c_int(T), c_int(E),
                                           c_int(top), _p(ids), _p(weights), self._stream()), "moe_topk")
 
-    def moe_route_softmax(self, h, w, correction, top, n_groups, keep, scale, ids, weights, logits):
+    def moe_route_scored(self, h, w, correction, top, ids, weights, logits, score, n_groups, keep, group_best, renorm, scale):
         self._on_gpu(h, w, correction, ids, weights, logits)
         T, E = logits.shape
         src, splits = self._product_sums(h, w, logits)
-        self._check(self.lib.hfb_moe_route_softmax(_p(src), c_int(splits), _p(correction), c_int(_dt(correction) if correction is not None else 0),
-                                                   c_int(T), c_int(E), c_int(top), c_int(n_groups), c_int(keep), c_float(scale), _p(ids),
-                                                   _p(weights), self._stream()), "moe_route_softmax")
+        self._check(self.lib.hfb_moe_route_scored(
+            _p(src), c_int(splits), _p(correction), c_int(_dt(correction) if correction is not None else 0), c_int(T), c_int(E), c_int(top),
+            c_int(score), c_int(n_groups), c_int(keep), c_int(group_best), c_int(1 if renorm else 0), c_float(scale), _p(ids), _p(weights),
+            self._stream()), "moe_route_scored")
 
     # ---- hyper-connections ----------------------------------------------------------------------------------
     def hc_spread(self, emb, x, S):
@@ -609,12 +623,12 @@ class NativeBackend:
                                            c_int(g_col0), c_int(gate), _p(out), c_int(_dt(out)), c_int(o.shape[0]), c_int(H), c_int(dv),
                                            self._stream()), "gate_norm")
 
-    def rotate_heads(self, src, splits, row, cos_sin, n_rot, positions, k_scale, q, k, u, H, d, dv):
+    def rotate_heads(self, src, splits, row, cos_sin, n_rot, positions, k_scale, q, k, u, H, d, dv, silu=False):
         self._on_gpu(src, cos_sin, positions, q, k, u)
         self._check(self.lib.hfb_rotate_heads(
             _p(src), c_int(splits), c_int(row), _p(cos_sin), c_int(n_rot), c_int(cos_sin.shape[0] if cos_sin is not None else 0), _p(positions),
             c_float(k_scale), _p(q), _p(k), _p(u), c_int(_dt(q)), c_int(q.shape[0]), c_int(H), c_int(d), c_int(dv), c_int(q.shape[1] // H),
-            c_int(u.shape[1] // H), self._stream()), "rotate_heads")
+            c_int(u.shape[1] // H), c_int(1 if silu else 0), self._stream()), "rotate_heads")
 
     def state_space_operands(self, src, splits, row, conv_w, conv_b, dt_bias, rate, carried, ctx, q, k, u, step, la, H, G, d, dv):
         self._on_gpu(src, conv_w, conv_b, dt_bias, rate, q, k, u, step, la, ctx.token_seq, ctx.cu_tokens, ctx.seq_slots)
@@ -647,12 +661,13 @@ class NativeBackend:
             _p(ctx.seq_slots), c_int(state.shape[0]), c_int(ctx.num_seqs), _p(o), c_int(H), c_int(Hq), c_int(d), c_int(dv), c_int(dp), c_int(dvp),
             self._stream()), "decay_walk")
 
-    def part_norm_gate(self, o, parts, eps, g, g_splits, g_stride, g_col0, w, gate_first, out):
+    def part_norm_gate(self, o, parts, eps, g, g_splits, g_stride, g_col0, w, gate_first, out, gate="silu"):
         self._on_gpu(o, g, w)
         self._rows_on_gpu(out)
         self._check(self.lib.hfb_part_norm_gate(
-            _p(o), _p(g), c_int(g_splits), c_int(g_stride), c_int(g_col0), _p(w), c_float(eps), c_int(1 if gate_first else 0), _p(out),
-            c_int(_dt(out)), c_int64(out.stride(0)), c_int(o.shape[0]), c_int(o.shape[1]), c_int(parts), self._stream()), "part_norm_gate")
+            _p(o), _p(g), c_int(g_splits), c_int(g_stride), c_int(g_col0), _p(w), c_float(eps), c_int(1 if gate_first else 0),
+            c_int(1 if gate == "sigmoid" else 0), _p(out), c_int(_dt(out)), c_int64(out.stride(0)), c_int(o.shape[0]), c_int(o.shape[1]),
+            c_int(parts), self._stream()), "part_norm_gate")
 
     def linear_row_norm_kv(self, a, w, buf, q_w, k_w, eps, slots, q_out, k_cache, v_cache, gate_out, H, G, d, dv):
         self._on_gpu(a, w, buf, q_w, k_w, slots, q_out, k_cache, v_cache, gate_out)
@@ -702,12 +717,12 @@ class NativeBackend:
         self._check(self.lib.hfb_moe_sort(_p(ids), c_int(ids.numel()), c_int(experts), c_int(tile), _p(order), _p(tile_expert),
                                           _p(tile_p0), _p(tile_n), _p(n_tiles), self._stream()), "moe_sort")
 
-    def moe_gemm(self, a, w, out, act, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles, max_tiles, tile):
+    def moe_gemm(self, a, w, out, act, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles, max_tiles, tile, clamp=None):
         self._on_gpu(a, w, out, order, tile_expert, tile_p0, tile_n, n_tiles)
-        MOE_TILE = tile
-        self._check(self.lib.hfb_moe_gemm(_p(a), c_int(_dt(a)), _p(w), c_int(_dt(w)), _p(out), c_int(_dt(out)), c_int(act),
+        consts = tuple(c_float(x) for x in (clamp or (0.0, 0.0, 0.0)))
+        self._check(self.lib.hfb_moe_gemm(_p(a), c_int(_dt(a)), _p(w), c_int(_dt(w)), _p(out), c_int(_dt(out)), c_int(act), *consts,
                                           c_int(w.shape[1]), c_int(w.shape[2]), _p(order), c_int(src_div), c_int(1 if scatter else 0),
-                                          _p(tile_expert), _p(tile_p0), _p(tile_n), _p(n_tiles), c_int(max_tiles), c_int(MOE_TILE),
+                                          _p(tile_expert), _p(tile_p0), _p(tile_n), _p(n_tiles), c_int(max_tiles), c_int(tile),
                                           self._stream()), "moe_gemm")
 
     def moe_combine(self, y, weights, out):

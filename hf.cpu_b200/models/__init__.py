@@ -57,6 +57,7 @@ class Model:
         p = self.plan
         self.positions = {name: make_part("position", spec) for name, spec in p.positions.items()}
         self.embedding = make_part("embedding", p.embedding)
+        self.transitions = {name: make_part("transition", spec) for name, spec in p.transitions.items()}
         self.layers: List[Layer] = []
         for ls in p.layers:
             self.layers.append(Layer(
@@ -76,6 +77,7 @@ class Model:
     def all_parts(self):
         yield self.embedding
         yield from self.positions.values()
+        yield from self.transitions.values()
         for l in self.layers:
             yield from l.parts()
         yield self.final_norm
@@ -114,6 +116,8 @@ class Model:
         total = self.head.weight_bytes() + self.final_norm.weight_bytes()
         for e in self.plan.schedule:
             total += sum(p.weight_bytes() for p in self.layers[e.layer].parts())
+            if e.enter is not None:
+                total += self.transitions[e.enter[0]].weight_bytes()
         return total
 
     # ---- forward ------------------------------------------------------------------------
@@ -129,6 +133,8 @@ class Model:
             with kernels.phase("glue"):
                 kernels.hc_spread(emb, x, S)
         schedule = self.plan.schedule
+        for tr in self.transitions.values():
+            tr.begin(ctx, x)
         xn = None                                # norm1 of the coming block, when the previous block computed it
         for i, e in enumerate(schedule):
             layer = self.layers[e.layer]
@@ -136,7 +142,16 @@ class Model:
             # the norm that follows this block: the next block's first, or, after the last block of a step whose
             # tokens all want their logits (a step of single tokens), the final norm
             extra = layer.post_norms()
-            if i + 1 < len(schedule):
+            if e.enter is not None:
+                # (what the block in front handed over is the transition's operand; the layer's input comes out of it)
+                out = ctx.buf("enter_xn", x.shape, self.run_dtype) if layer.block.state_spec() is None else None
+                done = self.transitions[e.enter[0]].enter(ctx, x, e.enter[1], xn, layer.norm1 if out is not None else None, out)
+                xn = out if done else None
+            if i + 1 < len(schedule) and schedule[i + 1].enter is not None:
+                next_norm = self.transitions[schedule[i + 1].enter[0]].operand_norm()
+                if getattr(layer.block, "wants_next_block", False):
+                    extra["next_block"] = None
+            elif i + 1 < len(schedule):
                 next_norm = self.layers[schedule[i + 1].layer].norm1
                 following = self.layers[schedule[i + 1].layer].block
                 if getattr(layer.block, "wants_next_block", False):

@@ -1,7 +1,7 @@
 """Interfaces of the parts a layer is put together from, and their registries.
 
-Five categories: ``norm``, ``position``, ``mixer``, ``ffn`` and ``block``.  A part
-is chosen by the ``kind`` of a :class:`PartSpec` and receives every size and
+Six categories of parts between embedding and head: ``norm``, ``position``, ``mixer``, ``ffn``, ``block`` and ``transition``
+(a step between layers).  A part is chosen by the ``kind`` of a :class:`PartSpec` and receives every size and
 constant through the spec's arguments; no part knows which model it is in.
 
 The reference runs one fixed layer with ``if`` switches for its variants
@@ -18,7 +18,7 @@ import torch
 from ..config.base import ConfigError, PartSpec
 from ..weights.loader import TensorSpec
 
-CATEGORIES = ("norm", "position", "mixer", "ffn", "block", "embedding", "head")
+CATEGORIES = ("norm", "position", "mixer", "ffn", "block", "embedding", "head", "transition")
 _REGISTRY: Dict[str, Dict[str, Callable[..., "Part"]]] = {c: {} for c in CATEGORIES}
 
 
@@ -180,4 +180,21 @@ class Block(Part):
         """Run one layer on the float32 residual stream ``x`` in place.  ``xn_ready`` is ``norm1(x)`` if the
         previous block already computed it.  If ``next_norm`` is given the block may return ``next_norm(x)`` of
         its result (computed in the tail of its last product); returning None leaves that norm to the next block."""
+        raise NotImplementedError
+
+
+class Transition(Part):
+    """A step on the stream right in front of a schedule entry (``ScheduleEntry.enter``)."""
+
+    def begin(self, ctx, x: torch.Tensor) -> None:
+        """Called once per step with the embedding output, before the first layer."""
+
+    def operand_norm(self) -> Optional[Norm]:
+        """What the block in front may hand over in place of the coming layer's normed input, or None."""
+        return None
+
+    def enter(self, ctx, x: torch.Tensor, number: int, ready: Optional[torch.Tensor], norm: Optional[Norm],
+              out: Optional[torch.Tensor]) -> bool:
+        """Change the stream ``x`` in place for pass ``number``; ``ready`` is ``operand_norm()`` of x if the block in front
+        made it.  With ``norm`` the step may also write ``out = norm(x)`` of its result; returns whether it did."""
         raise NotImplementedError

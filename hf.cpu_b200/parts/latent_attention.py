@@ -13,6 +13,11 @@ Per token, with h the mixer's input:
   of its key: ``score = ([Wuk_h^T q_plain | q_rot] . [c | r]) * scale``, ``out_h = Wuv_h (sum_j p_j c_j)``.
 * ``out = concat(out_h) W_o^T`` is added to the residual.
 
+Options: ``sink_tensor`` names a score per head without key and value that joins the softmax's denominator once (it is not
+scaled).  ``gate_tensor`` names an output gate, ``sigmoid(W_g h)`` per element of the concatenated heads: its rows stand
+behind the down projections' in the one product that reads h, the product's tail stores the sigmoids, and the value
+expansion multiplies by them where it stores its result.
+
 Where the cached row has a size the tiled tensor-core attention kernels take (they want value heads as wide as key
 heads), the whole row serves as the value: the rotated columns of the weighted sum are computed and not read.  Other
 sizes take the plain kernel, which reads a value as the first ``kv_rank`` elements of its key.
@@ -31,7 +36,7 @@ import torch
 
 from .. import kernels
 from ..config.base import UnsupportedError
-from ..weights.loader import TensorSpec, fused_rows
+from ..weights.loader import TensorSpec, fused_rows, pad_rows
 from .attention import OutputProduct
 from .base import CacheSpec, Mixer, register_part
 
@@ -41,7 +46,7 @@ class LatentAttention(OutputProduct, Mixer):
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, q_rank: int,
                  kv_rank: int, scale: float, norm_eps: float, window: int, position, prefix: str, positions=None,
-                 names=None, **_):
+                 names=None, sink_tensor=None, gate_tensor=None, **_):
         self.E, self.H, self.d, self.dr, self.dv = (int(hidden_size), int(num_heads), int(head_dim), int(rot_dim),
                                                     int(v_head_dim))
         self.Qr, self.R = int(q_rank), int(kv_rank)
@@ -60,6 +65,9 @@ class LatentAttention(OutputProduct, Mixer):
         n = {"dq": "dq", "dq_norm": "dq.norm", "uq": "uq", "dkv": "dkv", "dkv_norm": "dkv.norm", "uk": "uk", "uv": "uv", "o": "o"}
         n.update(names or {})
         self.names = {k: f"{prefix}.{v}" for k, v in n.items()}
+        self.sink_name = f"{prefix}.{sink_tensor}" if sink_tensor else None
+        self.gate_name = f"{prefix}.{gate_tensor}" if gate_tensor else None
+        self.sinks = None                               # float32 [H]
         self.w_down = self.w_uq = self.w_ukt = self.w_uv = self.w_o = self.b_o = None
         self.norm_q = self.norm_kv = None
 
@@ -74,7 +82,10 @@ class LatentAttention(OutputProduct, Mixer):
 
     def tensor_specs(self):
         n = self.names
-        return [TensorSpec(n["dq"], (self.Qr, self.E)), TensorSpec(n["dq_norm"], (self.Qr,), init="norm"),
+        s = [TensorSpec(self.sink_name, (self.H,))] if self.sink_name else []
+        if self.gate_name:
+            s.append(TensorSpec(self.gate_name, (self.H * self.dv, self.E)))
+        return s + [TensorSpec(n["dq"], (self.Qr, self.E)), TensorSpec(n["dq_norm"], (self.Qr,), init="norm"),
                 TensorSpec(n["uq"], (self.H * (self.d + self.dr), self.Qr)),
                 TensorSpec(n["dkv"], (self.R + self.dr, self.E)), TensorSpec(n["dkv_norm"], (self.R,), init="norm"),
                 TensorSpec(n["uk"], (self.H * self.d, self.R)), TensorSpec(n["uv"], (self.H * self.dv, self.R)),
@@ -82,18 +93,22 @@ class LatentAttention(OutputProduct, Mixer):
 
     def bind(self, tensors, run_dtype, device):
         n = self.names
-        # both down projections are one product: rows [query latent | key/value latent | rotated key part]
-        self.w_down = fused_rows(tensors, [n["dq"], n["dkv"]], device)
+        # both down projections are one product: rows [query latent | key/value latent | rotated key part (| output gate)]
+        self.w_down = fused_rows(tensors, [n["dq"], n["dkv"]] + ([self.gate_name] if self.gate_name else []), device)
+        if self.sink_name:
+            self.sinks = tensors[self.sink_name].to(torch.float32).contiguous()
         w_uq = tensors[n["uq"]].contiguous()
         if self.reorder:
             # "half" pairing: the rotated parts' rows into the order the kernels rotate in
             half = self.dr // 2
             order = torch.stack([torch.arange(half), torch.arange(half) + half], dim=1).reshape(-1).to(self.w_down.device)
-            tail = self.w_down[self.Qr + self.R:].clone()
-            self.w_down[self.Qr + self.R:] = tail[order]
+            part = slice(self.Qr + self.R, self.Qr + self.row)
+            self.w_down[part] = self.w_down[part].clone()[order]
             per_head = w_uq.reshape(self.H, self.d + self.dr, self.Qr).clone()
             per_head[:, self.d:] = per_head[:, self.d:][:, order.to(per_head.device)]
             w_uq = per_head.reshape(self.H * (self.d + self.dr), self.Qr).contiguous()
+        if self.gate_name:
+            self.w_down = pad_rows(self.w_down)
         self.norm_q = tensors[n["dq_norm"]].to(torch.float32).contiguous()
         self.norm_kv = tensors[n["dkv_norm"]].to(torch.float32).contiguous()
         self.w_uq = w_uq
@@ -124,10 +139,11 @@ class LatentAttention(OutputProduct, Mixer):
         cq = ctx.buf("lat_cq", (T, self.Qr), dt)
         q_plain = ctx.buf("lat_q_plain", (T, self.H * self.d), dt)
         q_att = ctx.buf("lat_q", (T, self.H * self.row), dt)
+        gate = ctx.buf("lat_gate", (T, self.H * self.dv), dt) if self.gate_name else None
         with kernels.phase("qkv"):
-            down = ctx.buf("lat_down32", (T, self.Qr + self.row), torch.float32)
+            down = ctx.buf("lat_down32", (T, self.w_down.shape[0]), torch.float32)
             kernels.linear_latent_split(xn, self.w_down, down, self.norm_q, self.norm_kv, self.eps, cos_sin, ctx.positions,
-                                        meta.slots, cq, cache.k, self.Qr, self.R, self.dr)
+                                        meta.slots, cq, cache.k, self.Qr, self.R, self.dr, gate_out=gate)
             q32 = ctx.buf("lat_q32", (T, self.H * (self.d + self.dr)), torch.float32)
             kernels.linear_latent_query_absorb(cq, self.w_uq, q32, cos_sin, ctx.positions, self.w_ukt, q_plain, q_att, self.H,
                                                self.d, self.dr)
@@ -137,13 +153,13 @@ class LatentAttention(OutputProduct, Mixer):
         with kernels.phase("attn"):
             if whole_row:
                 kernels.paged_attention(q_att, cache.k, cache.k, meta, ctx, self.H, 1, self.row, kernels.mask_code(self.window),
-                                        self.scale, lat, tiles=ctx.arrays(self.step_arrays_key()))
+                                        self.scale, lat, tiles=ctx.arrays(self.step_arrays_key()), sinks=self.sinks)
             else:
                 kernels.paged_attention(q_att, cache.k, None, meta, ctx, self.H, 1, self.row, kernels.mask_code(self.window),
-                                        self.scale, lat, dv=self.R, values_in_keys=True)
+                                        self.scale, lat, dv=self.R, values_in_keys=True, sinks=self.sinks)
         att = ctx.buf("lat_heads", (T, self.H * self.dv), dt)
         with kernels.phase("attn"):
-            kernels.headwise_linear(lat, self.w_uv, att, self.H, out_row, self.dv)
+            kernels.headwise_linear(lat, self.w_uv, att, self.H, out_row, self.dv, gate=gate)
         return att
 
 

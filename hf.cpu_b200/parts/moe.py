@@ -5,11 +5,14 @@ softmax over the chosen logits only.  Expert: ``Wd act(Wu x)`` (not gated, no bi
 chosen experts, plus, when the layer has one, a shared expert of the same form (with a width of its own) that every
 token runs.  (The reference has dense layers only.)
 
-Options: ``gated`` experts, ``Wd (act(Wg x) * (Wu x))``.  ``router`` "softmax_all": the scores are a softmax over all
-router outputs; an output is chosen by its score plus a stored ``correction`` (the weights use the score without it);
-the outputs form ``groups`` = (count, keep) equal groups of neighbours and only outputs of the ``keep`` groups with the
-largest choice score can be chosen; weights = scores of the chosen times ``route_scale``, not renormalised.  The last
-``identity`` router outputs are identity experts without tensors: their output is the layer's input itself.
+Options: ``gated`` experts, ``Wd (act(Wg x) * (Wu x))``, the shared expert then gated too; ``activation`` "clamped" with
+``clamp`` = {limit, alpha, offset} (and ``shared_clamp``) is the gated form of ``parts/ffn.py``.  Routers that score every
+output: "softmax_all" (a softmax over all router outputs) and "sigmoid" (each output by itself).  An output is chosen by
+its score plus a stored ``correction`` (the weights use the score without it); the outputs form ``groups`` = (count, keep)
+equal groups of neighbours, a group's score is the sum of its ``group_best`` (1 or 2) largest choice scores, and only
+outputs of the ``keep`` best groups can be chosen; weights = scores of the chosen, with ``renorm`` divided by their sum,
+times ``route_scale``.  The last ``identity`` router outputs are identity experts without tensors: their output is the
+layer's input itself.
 
 Nothing comes back to the host: the router's choices are grouped by expert on the device, the experts run as one
 grouped product over the groups' tiles (launch sizes are upper bounds), and each token's choices are summed in
@@ -31,29 +34,38 @@ class MoeFfn(FeedForward):
 
     def __init__(self, hidden_size: int, experts: int, top: int, expert_size: int, prefix: str, activation: str = "relu2",
                  router_bias: bool = True, shared_size: int = 0, names=None, gated: bool = False, router: str = "topk_softmax",
-                 correction=None, groups=None, identity: int = 0, route_scale: float = 1.0, **_):
+                 correction=None, groups=None, identity: int = 0, route_scale: float = 1.0, group_best: int = 1,
+                 renorm: bool = False, clamp=None, shared_clamp=None, **_):
         self.E, self.n, self.top, self.F, self.FS = int(hidden_size), int(experts), int(top), int(expert_size), int(shared_size or 0)
         self.gated, self.router, self.identity, self.route_scale = bool(gated), router, int(identity or 0), float(route_scale)
-        if router not in ("topk_softmax", "softmax_all"):
-            raise UnsupportedError(f"mixture of experts: router '{router}' is not known (topk_softmax, softmax_all)")
+        self.group_best, self.renorm = int(group_best), bool(renorm)
+        if router not in ("topk_softmax", "softmax_all", "sigmoid"):
+            raise UnsupportedError(f"mixture of experts: router '{router}' is not known (topk_softmax, softmax_all, sigmoid)")
         self.n_out = self.n + self.identity                 # router outputs: experts, then identity experts
         self.groups = (int(groups[0]), int(groups[1])) if groups else (1, 1)
-        if router == "topk_softmax" and (self.identity or groups or correction or self.route_scale != 1.0):
-            raise UnsupportedError("mixture of experts: identity experts, groups, a correction and a scale belong to the softmax_all router")
+        if router == "topk_softmax" and (self.identity or groups or correction or self.route_scale != 1.0 or self.renorm):
+            raise UnsupportedError("mixture of experts: identity experts, groups, a correction and a scale belong to the routers that "
+                                   "score every output")
+        if self.group_best not in (1, 2):
+            raise UnsupportedError("mixture of experts: a group is scored by its best one or its best two")
         if self.identity < 0 or self.n < 0 or self.n_out < 1:
             raise UnsupportedError(f"mixture of experts: {self.n} experts and {self.identity} identity experts")
         count, keep = self.groups
         if count < 1 or self.n_out % count or not 1 <= keep <= count or keep * (self.n_out // count) < self.top:
             raise UnsupportedError(f"mixture of experts: {count} groups of which {keep} are kept do not fit {self.n_out} router "
                                    f"outputs with top {self.top}")
-        if router_bias and router == "softmax_all":
-            raise UnsupportedError("mixture of experts: the softmax_all router has no bias")
+        if router_bias and router != "topk_softmax":
+            raise UnsupportedError("mixture of experts: a router that scores every output has no bias")
         self.correction_name = correction
         self.correction = None
         if not 1 <= self.top <= self.n_out:
             raise UnsupportedError(f"mixture of experts: top {self.top} of {self.n_out} experts")
-        if activation not in kernels.ACTIVATIONS:
+        if activation != "clamped" and activation not in kernels.ACTIVATIONS:
             raise UnsupportedError(f"mixture of experts: activation '{activation}' is not supported")
+        if (activation == "clamped") != bool(clamp) or (clamp and not self.gated) or bool(shared_clamp) != bool(clamp and self.FS):
+            raise UnsupportedError("mixture of experts: the clamped activation is gated, and its constants come with it")
+        consts = lambda c: (float(c["limit"]), float(c["alpha"]), float(c["offset"])) if c else None
+        self.clamp, self.shared_clamp = consts(clamp), consts(shared_clamp)
         self.activation, self.router_bias = activation, bool(router_bias)
         n = {"router": "router", "router_bias": "router.b", "expert": "e{}", "shared": "shared", "up": "up", "down": "down",
              "gate": "gate"}
@@ -76,6 +88,8 @@ class MoeFfn(FeedForward):
             s += [TensorSpec(self._expert(i, "up"), (self.F, self.E)), TensorSpec(self._expert(i, "down"), (self.E, self.F))]
         if self.FS:
             p = f"{self.prefix}.{self.nm['shared']}"
+            if self.gated:
+                s.append(TensorSpec(f"{p}.{self.nm['gate']}", (self.FS, self.E)))
             s += [TensorSpec(f"{p}.{self.nm['up']}", (self.FS, self.E)), TensorSpec(f"{p}.{self.nm['down']}", (self.E, self.FS))]
         return s
 
@@ -100,7 +114,11 @@ class MoeFfn(FeedForward):
         self.w_down = fused_rows(tensors, [self._expert(i, "down") for i in range(self.n)], device).view(self.n, self.E, self.F)
         if self.FS:
             p = f"{self.prefix}.{self.nm['shared']}"
-            self.ws_up = tensors[f"{p}.{self.nm['up']}"].contiguous()
+            if self.gated:
+                # (rows alternate gate, up, as the experts' do)
+                self.ws_up = fused_rows(tensors, [f"{p}.{self.nm['gate']}", f"{p}.{self.nm['up']}"], device, interleave=True)
+            else:
+                self.ws_up = tensors[f"{p}.{self.nm['up']}"].contiguous()
             self.ws_down = tensors[f"{p}.{self.nm['down']}"].contiguous()
 
     def weight_bytes(self):
@@ -111,7 +129,7 @@ class MoeFfn(FeedForward):
 
     def flops(self, rows):
         real = self.top * self.n / self.n_out             # chosen experts that are not identity experts, on average
-        return 2.0 * rows * (self.n_out * self.E + (3 if self.gated else 2) * real * self.E * self.F + 2 * self.E * self.FS)
+        return 2.0 * rows * (self.n_out * self.E + (3 if self.gated else 2) * self.E * (real * self.F + self.FS))
 
     def _experts(self, ctx, xn):
         """Router, grouping and the routed experts: (outputs of every (token, choice) [T * top, E] float32, weights [T, top])."""
@@ -121,9 +139,10 @@ class MoeFfn(FeedForward):
         wts = ctx.buf("moe_weights", (T, self.top), torch.float32)
         z = ctx.buf("moe_logits", (T, self.n_out), torch.float32)
         with kernels.phase("glue"):
-            if self.router == "softmax_all":
-                kernels.moe_route_softmax(xn, self.w_router, self.correction, self.top, self.groups[0], self.groups[1],
-                                          self.route_scale, ids, wts, z)
+            if self.router != "topk_softmax":
+                kernels.moe_route_scored(xn, self.w_router, self.correction, self.top, ids, wts, z,
+                                         score="sigmoid" if self.router == "sigmoid" else "softmax", n_groups=self.groups[0],
+                                         keep=self.groups[1], group_best=self.group_best, renorm=self.renorm, scale=self.route_scale)
             else:
                 kernels.moe_route(xn, self.w_router, self.b_router, self.top, ids, wts, z)
             mt = kernels.moe_max_tiles(P, self.n)
@@ -134,7 +153,8 @@ class MoeFfn(FeedForward):
         h = ctx.buf("moe_h", (P, self.F), xn.dtype)
         y = ctx.buf("moe_y", (P, self.E), xn.dtype if xn.dtype == torch.float32 else torch.float32)
         with kernels.phase("gate_up"):
-            kernels.moe_gemm(xn, self.w_up, h, self.activation, order, self.top, False, *tiles, n_tiles, P, glu=self.gated)
+            kernels.moe_gemm(xn, self.w_up, h, self.activation, order, self.top, False, *tiles, n_tiles, P, glu=self.gated,
+                             clamp=self.clamp)
         with kernels.phase("down"):
             kernels.moe_gemm(h, self.w_down, y, "none", order, 0, True, *tiles, n_tiles, P)
         if self.identity:
@@ -158,7 +178,11 @@ class MoeFfn(FeedForward):
     def _shared_hidden(self, ctx, xn):
         hs = ctx.buf("moe_hs", (xn.shape[0], self.FS), xn.dtype)
         with kernels.phase("gate_up"):
-            kernels.linear_act(xn, self.ws_up, hs, self.activation)
+            if self.gated:
+                gu = ctx.buf("moe_gate_up", (xn.shape[0], 2 * self.FS), xn.dtype)
+                kernels.linear_glu(xn, self.ws_up, gu, hs, self.activation, clamp=self.shared_clamp)
+            else:
+                kernels.linear_act(xn, self.ws_up, hs, self.activation)
         return hs
 
     def forward_into_norm(self, ctx, xn, y_buf, residual, post, next_norm, out):

@@ -17,16 +17,19 @@ class RmsNorm(Norm):
     weight (1 + w has more digits than bfloat16 keeps)."""
     graph_safe = True
 
-    def __init__(self, size: int, eps: float, tensor: str, offset: float = 0.0, **_):
+    def __init__(self, size: int, eps: float, tensor: str, offset: float = 0.0, optional: bool = False, **_):
         self.size, self.eps, self.tensor, self.offset = int(size), float(eps), tensor, float(offset)
+        self.optional = bool(optional)         # (a norm that nothing reads may be stored or not)
         self.weight = None
         self._w32 = None
 
     def tensor_specs(self):
         # random weights are drawn around the value that makes the norm's factor about one
-        return [TensorSpec(self.tensor, (self.size,), init="normal" if self.offset else "norm")]
+        return [TensorSpec(self.tensor, (self.size,), init="normal" if self.offset else "norm", optional=self.optional)]
 
     def bind(self, tensors, run_dtype, device):
+        if self.optional and self.tensor not in tensors:
+            return
         self.weight = tensors[self.tensor].contiguous()
         if self.offset:
             self.weight = (self.weight.to(torch.float32) + self.offset).contiguous()
@@ -44,6 +47,43 @@ class RmsNorm(Norm):
     def forward(self, x, out, rows=None):
         with kernels.phase("glue"):
             kernels.rmsnorm(x, self.weight, self.eps, out, rows)
+        return out
+
+    # ---- as the norm of a sublayer's output -------------------------------------------------------------
+    @staticmethod
+    def _tail(norm):
+        """``nxt`` of :func:`kernels.rms_tail` for the norm that follows, or None if that pass does not know it."""
+        if isinstance(norm, StreamCast):
+            return "copy"
+        return (norm.weight, norm.eps) if isinstance(norm, RmsNorm) else None
+
+    def add_into(self, y, residual, next_norm=None, out=None, mix=None):
+        """residual += norm(y (+ mix)); when ``next_norm`` is another RMSNorm (or the plain copy), ``out = next_norm(residual)``
+        comes out of the same pass.  Returns whether ``out`` was written.  ``mix`` = (rows, weights): a routed
+        feed-forward's chosen experts, summed by the same pass; y may then be None."""
+        nxt = self._tail(next_norm) if out is not None else None
+        with kernels.phase("glue"):
+            kernels.rms_tail(y, 1, residual, post=(self.weight, self.eps), nxt=nxt, out=out if nxt is not None else None, mix=mix)
+        return nxt is not None
+
+    def add_product_into(self, a, w, bias, y_buf, residual, next_norm=None, out=None, mix=None):
+        """The same for a sublayer whose output is a product, ``a @ w.T + bias (+ mix)``: where the product is split over
+        its inner dimension, the partial sums are summed by this norm's own pass."""
+        nxt = self._tail(next_norm) if out is not None else None
+        kernels.linear_rms_tail(a, w, y_buf, residual, bias=bias, post=(self.weight, self.eps), nxt=nxt,
+                                out=out if nxt is not None else None, mix=mix)
+        return nxt is not None
+
+
+class StreamCast(Norm):
+    """No norm at all: the stream in the run's type, for what reads it as it is.  Made by the parts that want it; not
+    registered."""
+
+    def forward(self, x, out, rows=None):
+        if rows is not None:
+            raise ValueError("the stream's copy takes every row")
+        with kernels.phase("glue"):
+            kernels.rms_tail(None, 0, x, nxt="copy", out=out)
         return out
 
 

@@ -315,11 +315,14 @@ class _ScalarDecay(_Recurrent):
 
 class Retention(_ScalarDecay):
     """Linear attention with a fixed decay per head and no softmax: q = Wq h and k = Wk h rotated (dimension i with i +
-    n_rot/2 of the leading n_rot), k times ``head_dim^(-1/2)``, u = v = Wv h, ``a`` the head's entry of ``decay``; every
-    head's o is divided by its root mean square (no weight), then multiplied by silu(Wg h), then ``Wo``."""
+    n_rot/2 of the leading n_rot), k times ``key_scale`` (None: ``head_dim^(-1/2)``), u = v = Wv h, ``a`` the head's entry of
+    ``decay``; every head's o is divided by its root mean square (no weight), then multiplied by silu(Wg h), then ``Wo``.
+    Options: ``activation`` "silu" on q, k and v (before any rotation); ``norm_tensor``: the heads are normed together, as one
+    row with that weight; ``gate`` "sigmoid".  Lightning attention is this mixer with silu, no rotation, keys as they are,
+    one norm over the row and a sigmoid gate (kind ``lightning_attention``)."""
 
     def __init__(self, hidden_size: int, num_heads: int, head_dim: int, v_head_dim: int, decay, norm_eps: float, prefix: str,
-                 position=None, positions=None, names=None, **_):
+                 position=None, positions=None, names=None, activation=None, key_scale=None, norm_tensor=None, gate: str = "silu", **_):
         self.E, self.H, self.d, self.dv = int(hidden_size), int(num_heads), int(head_dim), int(v_head_dim)
         self.eps, self.prefix = float(norm_eps), prefix
         self.decay = [float(a) for a in decay]
@@ -332,6 +335,12 @@ class Retention(_ScalarDecay):
             raise UnsupportedError(f"retention names position encoding '{position}', which the plan does not define")
         if self.rotary is not None and getattr(self.rotary, "pairing", "half") != "half":
             raise UnsupportedError("retention: the rotation pairs dimension i with i + n_rot/2")
+        if activation not in (None, "silu") or gate not in ("silu", "sigmoid"):
+            raise UnsupportedError(f"retention: activation '{activation}' or gate '{gate}' is not supported")
+        self.activation, self.gate = activation, gate
+        self.key_scale = self.d ** -0.5 if key_scale is None else float(key_scale)
+        self.norm_name = f"{prefix}.{norm_tensor}" if norm_tensor else None
+        self.norm_w = None
         n = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
         n.update(names or {})
         self.nm = n
@@ -342,12 +351,17 @@ class Retention(_ScalarDecay):
 
     def tensor_specs(self):
         KD, VD = self.H * self.d, self.H * self.dv
-        return [TensorSpec(self._t("q"), (KD, self.E)), TensorSpec(self._t("k"), (KD, self.E)), TensorSpec(self._t("v"), (VD, self.E)),
-                TensorSpec(self._t("g"), (VD, self.E)), TensorSpec(self._t("o"), (self.E, VD))]
+        s = [TensorSpec(self._t("q"), (KD, self.E)), TensorSpec(self._t("k"), (KD, self.E)), TensorSpec(self._t("v"), (VD, self.E)),
+             TensorSpec(self._t("g"), (VD, self.E)), TensorSpec(self._t("o"), (self.E, VD))]
+        if self.norm_name:
+            s.append(TensorSpec(self.norm_name, (VD,), init="norm"))
+        return s
 
     def bind(self, tensors, run_dtype, device):
         self.w_in = pad_rows(fused_rows(tensors, [self._t(x) for x in ("q", "k", "v", "g")], device))
         self.w_o = tensors[self._t("o")].contiguous()
+        if self.norm_name:
+            self.norm_w = tensors[self.norm_name].to(torch.float32).contiguous()
         # the logarithm in float64 from the configuration's numbers; a decay of zero as one that leaves nothing
         la = torch.tensor(self.decay, dtype=torch.float64).log().clamp_(min=-1e4)
         self.log_decay = la.to(torch.float32).to(device)
@@ -359,12 +373,14 @@ class Retention(_ScalarDecay):
         cos_sin, n_rot = (self.rotary.cos_sin, self.rotary.n_rot) if self.rotary is not None else (None, 0)
         with kernels.phase("qkv"):
             row, splits = kernels.product_sums(xn, self.w_in, ctx.buf("rec_in", (T, C), torch.float32))
-            kernels.rotate_heads(row, splits, C, cos_sin, n_rot, ctx.positions, self.d ** -0.5, q, k, u, self.H, self.d, self.dv)
+            kernels.rotate_heads(row, splits, C, cos_sin, n_rot, ctx.positions, self.key_scale, q, k, u, self.H, self.d, self.dv,
+                                 activation=self.activation)
         o = ctx.buf("rec_o", (T, VD), torch.float32)
         with kernels.phase("attn"):
             kernels.decay_scan(q, k, u, self.log_decay, None, None, self._matrix(state), ctx, o, self.H, self.H, self.d, self.dv,
                                chunks=ctx.arrays(self.ARRAYS))
-            kernels.part_norm_gate(o, self.H, self.eps, row, splits, C, 2 * KD + VD, None, False, out)
+            kernels.part_norm_gate(o, 1 if self.norm_name else self.H, self.eps, row, splits, C, 2 * KD + VD, self.norm_w, False, out,
+                                   gate=self.gate)
         return out
 
 
@@ -437,6 +453,7 @@ class Mamba2(_ScalarDecay):
 
 
 register_part("mixer", "retention", Retention)
+register_part("mixer", "lightning_attention", Retention)       # the same part under the name of the form with silu and one norm
 register_part("mixer", "mamba2", Mamba2)
 register_part("mixer", "gated_linear_attention", GatedLinearAttention)
 register_part("mixer", "mingru", MinGru)

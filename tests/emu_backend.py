@@ -154,6 +154,26 @@ class EmuBackend:
         self.linear(a, w, bias, y_buf, False)
         self.dyt_residual(y_buf, post, residual, nxt, out, mix=mix)
 
+    @staticmethod
+    def _rms(v, w, eps):
+        return v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps) * w.float()
+
+    def rms_tail(self, y, splits, residual, post, nxt, out, bias=None, mix=None, base=None):
+        M, E = residual.shape
+        if y is not None or mix is not None:
+            v = torch.zeros_like(residual)
+            if y is not None:
+                v = v + y.reshape(-1)[:splits * M * E].view(splits, M, E).sum(0)
+            if bias is not None:
+                v = v + bias.float()
+            if mix is not None:
+                v = v + (mix[1][:, :, None] * mix[0].view(M, -1, E)).sum(1)
+            if post is not None:
+                v = self._rms(v, *post)
+            residual.copy_((residual if base is None else base) + v)
+        if out is not None:
+            out.copy_((residual if nxt == "copy" else self._rms(residual, *nxt)).to(out.dtype))
+
     def linear_rope_norm_kv(self, a, w, bias, qkv_buf, cos_sin, n_rot, positions, slots, q_out, k_cache, v_cache, H, G, d, dv,
                             norm_eps, norm_weights=None, value_mix=None, pairing="half"):
         self.linear(a, w, bias, qkv_buf, False)
@@ -200,8 +220,12 @@ class EmuBackend:
         a, b = v[..., 0::2], v[..., 1::2]
         return torch.stack([a * c - b * s, a * s + b * c], -1).flatten(-2)
 
-    def linear_latent_split(self, a, w, buf, q_norm_w, kv_norm_w, eps, cos_sin, positions, slots, cq_out, cache, q_rank, kv_rank, rot):
+    def linear_latent_split(self, a, w, buf, q_norm_w, kv_norm_w, eps, cos_sin, positions, slots, cq_out, cache, q_rank, kv_rank, rot,
+                            gate_out=None):
         self.linear(a, w, None, buf, False)
+        if gate_out is not None:
+            gate_out.copy_(torch.sigmoid(buf[:, q_rank + kv_rank + rot:][:, :gate_out.shape[1]]).to(gate_out.dtype))
+            buf = buf[:, :q_rank + kv_rank + rot]
         unit = lambda v: v / torch.sqrt((v * v).mean(-1, keepdim=True) + eps)
         cq_out.copy_((unit(buf[:, :q_rank]) * q_norm_w).to(cq_out.dtype))
         c = unit(buf[:, q_rank:q_rank + kv_rank]) * kv_norm_w
@@ -221,9 +245,11 @@ class EmuBackend:
         if rot:
             q_att.view(T, H, -1)[..., att_col:att_col + rot] = self._rotate_pairs(q[..., d:], cos_sin, positions).to(q_att.dtype)
 
-    def headwise_linear(self, x, w, out, H, in_row, out_row):
+    def headwise_linear(self, x, w, out, H, in_row, out_row, gate=None):
         T, (_, N, K) = x.shape[0], w.shape
         y = torch.einsum("thk,hnk->thn", x.view(T, H, in_row)[..., :K].float(), w.float())
+        if gate is not None:
+            y = y * gate.view(T, H, N).float()
         out.view(T, H, out_row)[..., :N] = y.to(out.dtype)
 
     @staticmethod
@@ -268,22 +294,25 @@ class EmuBackend:
         ids.copy_(idx[:, :top].int())
         weights.copy_(torch.softmax(zc[:, :top], -1))
 
-    def moe_route_softmax(self, h, w, correction, top, n_groups, keep, scale, ids, weights, logits):
+    def moe_route_scored(self, h, w, correction, top, ids, weights, logits, score, n_groups, keep, group_best, renorm, scale):
         z = h.float() @ w.float().T
         logits.copy_(z)
-        s = torch.softmax(z, -1)
+        s = torch.sigmoid(z) if score == 1 else torch.softmax(z, -1)
         ch = s + correction.float() if correction is not None else s.clone()
         T, E = s.shape
         if n_groups > 1 and keep < n_groups:
             per = E // n_groups
-            best = ch.view(T, n_groups, per).max(-1).values
+            best = torch.sort(ch.view(T, n_groups, per), dim=-1, descending=True).values[..., :group_best].sum(-1)
             kept = torch.sort(best, dim=-1, descending=True, stable=True).indices[:, :keep]
             allow = torch.zeros(T, n_groups, dtype=torch.bool, device=s.device)
             allow.scatter_(1, kept, True)
             ch = torch.where(allow[:, :, None].expand(T, n_groups, per).reshape(T, E), ch, torch.full_like(ch, float("-inf")))
         idx = torch.sort(ch, dim=-1, descending=True, stable=True).indices[:, :top]
         ids.copy_(idx.int())
-        weights.copy_(torch.gather(s, 1, idx) * scale)
+        chosen = torch.gather(s, 1, idx)
+        if renorm:
+            chosen = chosen / (chosen.sum(-1, keepdim=True) + 1e-20)
+        weights.copy_(chosen * scale)
 
     def product_sums(self, a, w, buf, finished=False):
         self.linear(a, w, None, buf, False)
@@ -425,9 +454,11 @@ class EmuBackend:
         d.zero_()
         d[..., :x.shape[-1]] = x.to(dst.dtype)
 
-    def rotate_heads(self, src, splits, row, cos_sin, n_rot, positions, k_scale, q, k, u, H, d, dv):
+    def rotate_heads(self, src, splits, row, cos_sin, n_rot, positions, k_scale, q, k, u, H, d, dv, silu=False):
         T = q.shape[0]
         r = src.reshape(-1)[:splits * T * row].view(splits, T, row).sum(0)
+        if silu:
+            r = r * torch.sigmoid(r)
         qk = r[:, :2 * H * d].view(T, 2 * H, d).clone()
         if n_rot:
             half = n_rot // 2
@@ -478,10 +509,11 @@ class EmuBackend:
                 o[t] = y[:, :dv].reshape(-1)
             state[slots[s]] = S
 
-    def part_norm_gate(self, o, parts, eps, g, g_splits, g_stride, g_col0, w, gate_first, out):
+    def part_norm_gate(self, o, parts, eps, g, g_splits, g_stride, g_col0, w, gate_first, out, gate="silu"):
         T, C = o.shape
+        kind = gate
         z = g.reshape(-1)[:g_splits * T * g_stride].view(g_splits, T, g_stride).sum(0)[:, g_col0:g_col0 + C]
-        gate = z * torch.sigmoid(z)
+        gate = torch.sigmoid(z) if kind == "sigmoid" else z * torch.sigmoid(z)
         y = o * gate if gate_first else o
         p = y.view(T, parts, -1)
         y = (p / torch.sqrt((p * p).mean(-1, keepdim=True) + eps)).reshape(T, C)
@@ -523,7 +555,8 @@ class EmuBackend:
             at += c
         n_tiles[0] = n
 
-    def moe_gemm(self, a, w, out, act, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles, max_tiles, tile):
+    def moe_gemm(self, a, w, out, act, order, src_div, scatter, tile_expert, tile_p0, tile_n, n_tiles, max_tiles, tile,
+                 clamp=None):
         assert int(n_tiles[0]) <= max_tiles
         for i in range(int(n_tiles[0])):
             e, p0, n = int(tile_expert[i]), int(tile_p0[i]), int(tile_n[i])
@@ -532,7 +565,11 @@ class EmuBackend:
             src = pairs // src_div if src_div else places
             dst = pairs if scatter else places
             z = a[src].float() @ w[e].float().T
-            if act >> 8:
+            if clamp is not None:
+                limit, alpha, offset = clamp
+                g, u = z[:, 0::2].clamp(max=limit), z[:, 1::2].clamp(-limit, limit)
+                out[dst] = (g * torch.sigmoid(alpha * g) * (u + offset)).to(out.dtype)
+            elif act >> 8:
                 out[dst] = (self._activate(z[:, 0::2], act & 255) * z[:, 1::2]).to(out.dtype)
             else:
                 out[dst] = self._activate(z, act).to(out.dtype)

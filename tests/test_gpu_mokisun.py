@@ -514,7 +514,8 @@ def test_softmax_router_with_groups_and_correction(dtype, r_cfg):
     ids = torch.empty(T, top, dtype=torch.int32, device=DEV)
     wts = torch.empty(T, top, device=DEV)
     logits = torch.empty(T, n_all, device=DEV)
-    K().moe_route_softmax(h, w, dev(corr), top, groups[0] if groups else 1, groups[1] if groups else 1, 1.7, ids, wts, logits)
+    K().moe_route_scored(h, w, dev(corr), top, ids, wts, logits, n_groups=groups[0] if groups else 1, keep=groups[1] if groups else 1,
+                         scale=1.7)
     assert rel(logits, f64(h) @ f64(w).T) < 1e-5
     # rows on which the choice is close in the plain implementation may differ in order; no row may differ in its set by
     # more than a close call
