@@ -305,11 +305,13 @@ state_space_operands_kernel(const float *src, int splits, int row_stride, const 
 
 // ---- the walk ---------------------------------------------------------------------------------------------------
 // L lanes share a column of S, each holding J vectors of four of its entries; a group of L lanes takes DS_COLS columns.
+// Where the decay is the same for every token, `fixed` [H] holds it as it is: an exponential made from its rounded logarithm
+// may be off by an ulp, the same way at every token, and a thousand tokens add that up.
 constexpr int DS_COLS = 4;
 
 template <typename TI, int L, int J>
 __global__ void __launch_bounds__(128)
-decay_walk_kernel(const TI *q, const TI *k, const TI *u, const float *la, int la_stride, const float *step, const float *skip,
+decay_walk_kernel(const TI *q, const TI *k, const TI *u, const float *la, int la_stride, const float *fixed, const float *step, const float *skip,
                   float *state, size_t slot_stride, const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, float *o, int H,
                   int Hq, int dp, int dv, int dvp, int *err)
 {
@@ -330,7 +332,7 @@ decay_walk_kernel(const TI *q, const TI *k, const TI *u, const float *la, int la
             const int i = (part + j * L) * 4;
             S[c][j] = (c0 + c < dvp && i < dp) ? *(const float4 *)(sp + (size_t)(c0 + c) * dp + i) : zero;
         }
-    const float dsk = skip ? skip[h] : 0.f;
+    const float dsk = skip ? skip[h] : 0.f, a_fixed = fixed ? fixed[h] : 0.f;
     float4 qn[J], kn[J];
     float un[DS_COLS], an, cn;
     auto fetch = [&](int t) {
@@ -354,7 +356,7 @@ decay_walk_kernel(const TI *q, const TI *k, const TI *u, const float *la, int la
         for (int j = 0; j < J; j++) { qa[j] = qn[j]; ka[j] = kn[j]; }
 #pragma unroll
         for (int c = 0; c < DS_COLS; c++) ua[c] = un[c];
-        const float a = expf(an), cs = cn;
+        const float a = fixed ? a_fixed : expf(an), cs = cn;
         if (t + 1 < t1) fetch(t + 1);
         float dot[DS_COLS];
 #pragma unroll
@@ -897,8 +899,8 @@ extern "C" int hfb_state_space_operands(const float *src, int splits, int row_st
     return hfb_conv_carry(src, splits, row_stride, H * dv, taps, carried, slot_stride, cu_tokens, seq_slots, n_slots, S, T, CC, s);
 }
 
-extern "C" int hfb_decay_walk(const void *q, const void *k, const void *u, int dt, const float *la, int la_stride, const float *step,
-                              const float *skip, float *state, int64_t slot_stride, const int32_t *cu_tokens, const int32_t *seq_slots,
+extern "C" int hfb_decay_walk(const void *q, const void *k, const void *u, int dt, const float *la, int la_stride, const float *fixed,
+                              const float *step, const float *skip, float *state, int64_t slot_stride, const int32_t *cu_tokens, const int32_t *seq_slots,
                               int n_slots, int S, float *o, int H, int Hq, int d, int dv, int dp, int dvp, hfb_stream s)
 {
     if (S <= 0) return HFB_OK;
@@ -910,7 +912,7 @@ extern "C" int hfb_decay_walk(const void *q, const void *k, const void *u, int d
 #define HFB_WALK(TY, L, J) do { \
         const int cols = 4 * (32 / L) * DS_COLS; \
         g_launch_err = launch_pdl(decay_walk_kernel<TY, L, J>, dim3(S, H, (dvp + cols - 1) / cols), dim3(128), 0, (cudaStream_t)s, (const TY *)q, \
-            (const TY *)k, (const TY *)u, la, la_stride, step, skip, state, (size_t)slot_stride, cu_tokens, seq_slots, n_slots, o, H, Hq, dp, dv, dvp, \
+            (const TY *)k, (const TY *)u, la, la_stride, fixed, step, skip, state, (size_t)slot_stride, cu_tokens, seq_slots, n_slots, o, H, Hq, dp, dv, dvp, \
             error_word()); \
     } while (0)
 #define HFB_WALKS(TY) do { \

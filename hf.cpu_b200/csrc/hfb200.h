@@ -353,7 +353,7 @@ int hfb_conv_carry(const float *x, int splits, int x_stride, int x_col0, int tap
  *   i + n_rot / 2), keys times k_scale.
  * state_space_operands: q, k, u, step, la from rows [z: H dv | x: H dv | B: G d | C: G d | dt: H | ..]: x, B, C through a
  *   causal convolution with bias and silu (carried inputs as in conv_carry), step = softplus(dt + dt_bias), la = -rate step.
- * decay_walk: token by token.  decay_chunks: chunks of hfb_decay_chunk_tokens() tokens, bfloat16 operands.
+ * decay_walk: token by token; fixed [H]: exp(la) itself where it is the same for every token (null: made from la).  decay_chunks: chunks of hfb_decay_chunk_tokens() tokens, bfloat16 operands.
  * part_norm_gate: rows of o in `parts` equal parts, each divided by its root mean square; silu(g), or sigmoid(g) (sigmoid != 0),
  *   multiplies before (gate_first) or after; times w [C] where given; rows of out out_stride elements apart. */
 int hfb_rotate_heads(const float *src, int splits, int row_stride, const float *cos_sin, int n_rot, int n_positions,
@@ -364,8 +364,8 @@ int hfb_state_space_operands(const float *src, int splits, int row_stride, const
                              const int32_t *token_seq, const int32_t *cu_tokens, const int32_t *seq_slots, int n_slots, int S,
                              void *q, void *k, void *u, int out_dt, float *step, float *la, int T, int H, int G, int d, int dv,
                              int dp, int dvp, hfb_stream s);
-int hfb_decay_walk(const void *q, const void *k, const void *u, int dt, const float *la, int la_stride, const float *step,
-                   const float *skip, float *state, int64_t slot_stride, const int32_t *cu_tokens, const int32_t *seq_slots,
+int hfb_decay_walk(const void *q, const void *k, const void *u, int dt, const float *la, int la_stride, const float *fixed,
+                   const float *step, const float *skip, float *state, int64_t slot_stride, const int32_t *cu_tokens, const int32_t *seq_slots,
                    int n_slots, int S, float *o, int H, int Hq, int d, int dv, int dp, int dvp, hfb_stream s);
 int hfb_decay_chunk_tokens(void);
 size_t hfb_decay_chunks_scratch(int chunks, int H, int dp, int dvp);

@@ -814,12 +814,14 @@ def state_space_operands(src, splits: int, row: int, conv_w, conv_b, dt_bias, ra
                                    int(d), int(dv))
 
 
-def decay_scan(q, k, u, la, step, skip, state, ctx, o, H: int, Hq: int, d: int, dv: int, chunks=None) -> None:
+def decay_scan(q, k, u, la, step, skip, state, ctx, o, H: int, Hq: int, d: int, dv: int, chunks=None, fixed=None) -> None:
     """Per head, along each request's tokens from its slot's state: S <- exp(la) S + step k u^T, o = S^T q + skip u.  q, k [T,
     Hq heads], u [T, H heads] with heads padded with zeros to :func:`padded_head`; ``la`` float32 [T, H], or [H] for a decay
     that is the same for every token; ``step`` float32 [T, H] or None (1); ``skip`` float32 [H] or None; ``state`` float32
     [slots, H, padded dv, padded d]; ``o`` float32 [T, H * dv].  ``chunks``: the device arrays of :func:`decay_chunk_arrays`
-    for this step (empty or None: the walk)."""
+    for this step (empty or None: the walk).  ``fixed`` (float32 [H]): exp(la) itself, where it is the same for every token;
+    the walk then uses it as it is."""
+    _need(fixed is None or (fixed.shape == la.shape == (H,) and fixed.dtype == torch.float32), "decay_scan: fixed decays are float32 [H], as la is")
     _decay_ok(q, k, u, H, Hq, d, dv, "decay_scan")
     T, dp, dvp = q.shape[0], padded_head(d), padded_head(dv)
     _need(la.dtype == torch.float32 and la.shape in ((T, H), (H,)), "decay_scan: la is float32 [T, H] or [H]")
@@ -828,7 +830,8 @@ def decay_scan(q, k, u, la, step, skip, state, ctx, o, H: int, Hq: int, d: int, 
     _need(state.dtype == torch.float32 and state.shape[1:] == (H, dvp, dp) and state.stride()[1:] == (dvp * dp, dp, 1)
           and state.stride(0) % 4 == 0, "decay_scan: state is float32 [slots, H, padded dv, padded d], slots a multiple of four apart")
     _need(o.shape == (T, H * dv) and o.dtype == torch.float32, "decay_scan: o is float32 [T, H * dv]")
-    backend().decay_scan(q, k, u, la, step, skip, state, ctx, o, int(H), int(Hq), int(d), int(dv), chunks or {})
+    backend().decay_scan(q, k, u, la, step, skip, state, ctx, o, int(H), int(Hq), int(d), int(dv), chunks or {},
+                         **({"fixed": fixed} if fixed is not None else {}))
 
 
 def part_norm_gate(o, parts: int, eps: float, g, g_splits: int, g_stride: int, g_col0: int, w, gate_first: bool, out,

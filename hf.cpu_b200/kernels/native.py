@@ -641,8 +641,8 @@ class NativeBackend:
         if taps > 1 and q.shape[0] != ctx.num_seqs:
             self.launches += 1
 
-    def decay_scan(self, q, k, u, la, step, skip, state, ctx, o, H, Hq, d, dv, chunks):
-        self._on_gpu(q, k, u, la, step, skip, o, ctx.cu_tokens, ctx.seq_slots)
+    def decay_scan(self, q, k, u, la, step, skip, state, ctx, o, H, Hq, d, dv, chunks, fixed=None):
+        self._on_gpu(q, k, u, la, fixed, step, skip, o, ctx.cu_tokens, ctx.seq_slots)
         dp, dvp = q.shape[1] // Hq, u.shape[1] // H
         la_stride = H if la.dim() == 2 else 0
         if chunks and self.decay_chunks and q.dtype == torch.bfloat16:
@@ -657,7 +657,7 @@ class NativeBackend:
                 self.launches += 2
                 return
         self._check(self.lib.hfb_decay_walk(
-            _p(q), _p(k), _p(u), c_int(_dt(q)), _p(la), c_int(la_stride), _p(step), _p(skip), _p(state), c_int64(state.stride(0)), _p(ctx.cu_tokens),
+            _p(q), _p(k), _p(u), c_int(_dt(q)), _p(la), c_int(la_stride), _p(fixed), _p(step), _p(skip), _p(state), c_int64(state.stride(0)), _p(ctx.cu_tokens),
             _p(ctx.seq_slots), c_int(state.shape[0]), c_int(ctx.num_seqs), _p(o), c_int(H), c_int(Hq), c_int(d), c_int(dv), c_int(dp), c_int(dvp),
             self._stream()), "decay_walk")
 

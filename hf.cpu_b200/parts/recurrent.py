@@ -344,7 +344,7 @@ class Retention(_ScalarDecay):
         n = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o"}
         n.update(names or {})
         self.nm = n
-        self.w_in = self.w_o = self.log_decay = None
+        self.w_in = self.w_o = self.log_decay = self.decays = None
 
     def state_spec(self):
         return StateSpec((self.n_matrix,))
@@ -362,8 +362,10 @@ class Retention(_ScalarDecay):
         self.w_o = tensors[self._t("o")].contiguous()
         if self.norm_name:
             self.norm_w = tensors[self.norm_name].to(torch.float32).contiguous()
-        # the logarithm in float64 from the configuration's numbers; a decay of zero as one that leaves nothing
-        la = torch.tensor(self.decay, dtype=torch.float64).log().clamp_(min=-1e4)
+        # the decays themselves for the walk; for the chunks their logarithms, made in float64 (of a decay of zero: one that
+        # leaves nothing)
+        self.decays = torch.tensor(self.decay, dtype=torch.float32).to(device)
+        la = self.decays.cpu().double().log().clamp_(min=-1e4)
         self.log_decay = la.to(torch.float32).to(device)
 
     def operand(self, ctx, xn, cache, state, write_cache, out):
@@ -378,7 +380,7 @@ class Retention(_ScalarDecay):
         o = ctx.buf("rec_o", (T, VD), torch.float32)
         with kernels.phase("attn"):
             kernels.decay_scan(q, k, u, self.log_decay, None, None, self._matrix(state), ctx, o, self.H, self.H, self.d, self.dv,
-                               chunks=ctx.arrays(self.ARRAYS))
+                               chunks=ctx.arrays(self.ARRAYS), fixed=self.decays)
             kernels.part_norm_gate(o, 1 if self.norm_name else self.H, self.eps, row, splits, C, 2 * KD + VD, self.norm_w, False, out,
                                    gate=self.gate)
         return out

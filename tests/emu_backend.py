@@ -490,13 +490,13 @@ class EmuBackend:
         step.copy_(torch.nn.functional.softplus(r[:, inner + C:inner + C + H] + dt_bias.float()))
         la.copy_(-rate * step)
 
-    def decay_scan(self, q, k, u, la, step, skip, state, ctx, o, H, Hq, d, dv, chunks):
+    def decay_scan(self, q, k, u, la, step, skip, state, ctx, o, H, Hq, d, dv, chunks, fixed=None):
         T = q.shape[0]
         rep = H // Hq
         qh = q.float().view(T, Hq, -1).repeat_interleave(rep, 1)
         kh = k.float().view(T, Hq, -1).repeat_interleave(rep, 1)
         uh = u.float().view(T, H, -1)
-        a = torch.exp(la).expand(T, H)
+        a = (torch.exp(la) if fixed is None else fixed).expand(T, H)
         cu, slots = ctx.cu_tokens.tolist(), ctx.seq_slots.tolist()
         for s in range(len(slots)):
             S = state[slots[s]].clone()                                        # [H, dvp, dp]
