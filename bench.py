@@ -365,11 +365,45 @@ def tupalorn_configs(z):
     return tupalorn, silupel_configs(z)[0]
 
 
+# ---- `--compare birizen`: the Birizen design beside the Manapel design at equal layer sizes --------------------------
+# Four stored layers, lightning attention and latent attention in turn, the first two of which run three times (eight layer
+# runs, three entries into the loop); every layer with gated routed experts, eight groups of which half are kept, and a
+# shared expert.  The latent row (kv_rank + rot_dim) is 128.  The Manapel twin has eight layers of attention with as many
+# heads of the same size, routed experts and a shared one with as many weights per token (not gated: 2 F' = 3 F).
+BIRIZEN_SIZES = {
+    "w1024_h64": dict(width=1024, heads=16, kv=4, dim=64, rot=32, q_rank=384, kv_rank=96, rot_dim=32, ldim=64, experts=16, top=2, ff=384,
+                      shared=768, groups=(4, 2), vocab=32768),
+    "w2048_h128": dict(width=2048, heads=16, kv=4, dim=128, rot=64, q_rank=768, kv_rank=96, rot_dim=32, ldim=128, experts=32, top=4, ff=768,
+                       shared=1536, groups=(8, 4), vocab=32768),
+    "w4096_h128": dict(width=4096, heads=32, kv=8, dim=128, rot=128, q_rank=1536, kv_rank=96, rot_dim=32, ldim=128, experts=32, top=4, ff=1536,
+                       shared=3072, groups=(8, 4), vocab=32768),
+}
+
+
+def birizen_configs(z):
+    n = z["width"] // z["ldim"]
+    lightning = dict(type="lightning", mixer=dict(heads=n, dim=z["ldim"], vdim=z["ldim"], decay=[1.0 - 2.0 ** (-5.0 - 4.0 * i / n) for i in range(n)]))
+    latent = dict(type="latent_attention", mixer=dict(
+        heads=z["heads"], dim=z["dim"], rot_dim=z["rot_dim"], vdim=z["dim"], q_rank=z["q_rank"], kv_rank=z["kv_rank"],
+        scale=(z["dim"] + z["rot_dim"]) ** -0.5,
+        rot=dict(dims=z["rot_dim"], base=10000.0, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0))))
+    mlp = dict(kind="moe", expert=dict(ff=z["ff"], limit=7.0), shared=dict(ff=z["shared"], limit=7.0),
+               router=dict(experts=z["experts"], top=z["top"], groups=dict(count=z["groups"][0], keep=z["groups"][1])))
+    birizen = dict(architecture="Birizen", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), max_positions=8192,
+                   layers=[dict((lightning, latent)[i % 2], mlp=mlp) for i in range(4)], loop=dict(start=0, stop=2, times=3))
+    m_att = dict(heads=z["heads"], kv_heads=z["kv"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5, rot=dict(dims=z["rot"], base=10000.0))
+    m_moe = dict(kind="moe", router=dict(experts=z["experts"], top=z["top"]), expert=dict(ff=3 * z["ff"] // 2), shared=dict(ff=3 * z["shared"] // 2))
+    manapel = dict(architecture="Manapel", vocab=z["vocab"], width=z["width"], logit_scale=1.0, norm=dict(eps=1e-5), max_positions=8192,
+                   layers=[dict(type="attention", mixer=m_att, mlp=m_moe) for _ in range(8)])
+    return birizen, manapel
+
+
 COMPARISONS = {"manapel": (COMPARE_SIZES, compare_configs), "peludra": (PELUDRA_SIZES, peludra_configs),
                "mokisun": (MOKISUN_SIZES, mokisun_configs), "silupel": (SILUPEL_SIZES, silupel_configs),
-               "tupalorn": (TUPALORN_SIZES, tupalorn_configs)}
+               "tupalorn": (TUPALORN_SIZES, tupalorn_configs), "birizen": (BIRIZEN_SIZES, birizen_configs)}
 # the design each comparison stands beside
-TWINS = {"manapel": "qwen2", "peludra": "qwen2", "mokisun": "manapel", "silupel": "peludra", "tupalorn": "silupel"}
+TWINS = {"manapel": "qwen2", "peludra": "qwen2", "mokisun": "manapel", "silupel": "peludra", "tupalorn": "silupel",
+         "birizen": "manapel"}
 
 
 def phase_work(model, q_len, ctx_len, batch):
@@ -379,7 +413,7 @@ def phase_work(model, q_len, ctx_len, batch):
     weights the choices are close to uniform, so n (1 - (1 - 1/n)^(T top)) of n experts are expected to be chosen."""
     T = batch * q_len
     el = 2
-    work = {k: [0.0, 0.0] for k in ("qkv", "attn", "wo", "gate_up", "down", "head")}
+    work = {k: [0.0, 0.0] for k in ("qkv", "attn", "wo", "gate_up", "down", "join", "head")}
 
     def add(k, ops, nbytes):
         work[k][0] += ops
@@ -454,6 +488,10 @@ def phase_work(model, q_len, ctx_len, batch):
         L = model.layers[e.layer]
         f = L.ffn
         before = list(work["wo"])
+        if e.enter is not None:
+            # the product with the stream, its share of the product with the embedding, and the pass over the stream
+            tr = model.transitions[e.enter[0]]
+            add("join", tr.flops(T), tr.weight_bytes() + T * tr.E * (el + 4 + 4 + 4 + el))
         mixer(L.mixer)
         if getattr(L.block, "widths", None) is not None:
             # one product ends both sublayers; its time is the feed-forward's down phase
@@ -659,7 +697,7 @@ def main():
     ap.add_argument("--workload", choices=sorted(WORKLOADS), help="run one of the other sized workloads end to end through "
                     "Session.generate instead of the record (c3: 0.5B sizes, mixed chunked prompts and decodes; c4: 32B sizes)")
     ap.add_argument("--compare", choices=sorted(COMPARISONS), help="instead of the record: prefill and decode of that design beside the "
-                    "design closest to it (the Qwen2 decoder; for mokisun, Manapel) at equal layer sizes (random weights), one JSON line per size "
+                    "design closest to it (the Qwen2 decoder; for mokisun and birizen, Manapel) at equal layer sizes (random weights), one JSON line per size "
                     "and architecture")
     ap.add_argument("--sizes", default="", help="with --compare: the sizes to run, with commas (default: all)")
     ap.add_argument("--ref-layers", type=int, default=28, help="layers the reference arm runs (it is a CPU program)")
