@@ -497,7 +497,7 @@ def phase_work(model, q_len, ctx_len, batch):
             # one product ends both sublayers; its time is the feed-forward's down phase
             add("down", work["wo"][0] - before[0], work["wo"][1] - before[1] - 4 * T * f.E)
             work["wo"] = before
-        if hasattr(f, "w_up"):
+        if hasattr(f, "w_up") and not hasattr(f, "w_router"):
             add("gate_up", 2.0 * T * f.w_up.numel(), el * (f.w_up.numel() + T * (f.E + f.F)))
             add("down", 2.0 * T * f.w_down.numel(), el * (f.w_down.numel() + T * f.F) + 4 * T * f.E)
         elif hasattr(f, "w_gate_up"):

@@ -64,6 +64,8 @@ struct AttnParams {
     // score <- softcap * tanh(score / softcap), applied after the factors and before bias and softmax (0: none)
     const float *head_scales = nullptr;
     float softcap = 0.f, scale = 0.f;   // scale: the plain factor (scale_log2 without log2(e)), for the capped form
+    // the decode kernel: neighbouring groups of heads that read the same key/value head (G counts the groups)
+    int kv_share = 1;
 };
 
 // Byte offset of 16-byte chunk `c` of row `row` in a tile whose rows hold D bf16 (D = 64 or 128).

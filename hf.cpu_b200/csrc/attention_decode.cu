@@ -89,7 +89,7 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
         // The lanes look up 32 pages at a time (the pages of several tiles, one coalesced read of the block
         // table); lane 0 then asks for tile after tile without waiting for another table entry.
         const int32_t *table = p.block_table + (size_t)seq * p.max_blocks;
-        const int bs = p.block_size, pages = ABN / bs, tiles_per_round = 32 / pages;
+        const int bs = p.block_size, pages = ABN / bs, tiles_per_round = 32 / pages, kv_g = g / p.kv_share;
         bool waited = false;
         for (int kt0 = kt_lo; kt0 < kt_hi; kt0 += tiles_per_round) {
             const int key0 = kt0 * ABN + lane * bs, blk = key0 / bs;
@@ -114,10 +114,10 @@ attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __g
                     if (lane == 0) {
                         const uint32_t dst = st0 + (uint32_t)s * 2 * TILE + (uint32_t)pg * 2 * page_bytes;
                         if (ONE_MAP) {
-                            tma_load_4d(dst, &map_k, 0, row, g * HALVES, 0, full0 + 8 * s);
+                            tma_load_4d(dst, &map_k, 0, row, kv_g * HALVES, 0, full0 + 8 * s);
                         } else {
-                            tma_load_3d(dst, &map_k, 0, row, g * HALVES, full0 + 8 * s);
-                            tma_load_3d(dst + page_bytes, &map_v, 0, row, g * HALVES, full0 + 8 * s);
+                            tma_load_3d(dst, &map_k, 0, row, kv_g * HALVES, full0 + 8 * s);
+                            tma_load_3d(dst + page_bytes, &map_v, 0, row, kv_g * HALVES, full0 + 8 * s);
                         }
                     }
                 }
@@ -460,7 +460,12 @@ extern "C" int hfb_attention_decode_opt(const void *q, const void *k_cache, cons
 {
     if (n_tiles <= 0) return HFB_OK;
     if (d != 64 && d != 128) return fail(HFB_ENOTSUP, "attention_decode: head_dim %d (64 and 128 only)", d);
-    if (G <= 0 || H % G || H / G > 16) return fail(HFB_ENOTSUP, "attention_decode: %d heads over %d key/value heads do not fit 16 rows", H, G);
+    if (G <= 0 || H % G) return fail(HFB_ENOTSUP, "attention_decode: %d heads over %d key/value heads", H, G);
+    // more heads on a key/value head than a tile has rows: as several groups that read the same keys and values
+    const int kv_heads = G;
+    int share = 1;
+    while (H / G > 16 * share || (H / G) % share) share++;
+    G *= share;
     if (block_size < 8 || block_size > ABN || ABN % block_size) return fail(HFB_ENOTSUP, "attention_decode: block size %d (8..64, dividing 64)", block_size);
     if (num_pages * block_size >= (1ll << 31) - ABN) return fail(HFB_ENOTSUP, "attention_decode: cache too large for 32-bit coordinates");
     if (((uintptr_t)q & 15) || ((uintptr_t)k_cache & 15) || ((uintptr_t)v_cache & 15))
@@ -472,14 +477,14 @@ extern "C" int hfb_attention_decode_opt(const void *q, const void *k_cache, cons
     bool one_map = false;
     int rc;
     const int slots = (int)(num_pages * block_size);
-    if ((rc = tensor_map_kv(k_cache, v_cache, slots, G * d, block_size, d / 64, maps, &one_map)) != HFB_OK) return rc;
+    if ((rc = tensor_map_kv(k_cache, v_cache, slots, kv_heads * d, block_size, d / 64, maps, &one_map)) != HFB_OK) return rc;
     const CUtensorMap &mk = maps[0], &mv = maps[one_map ? 0 : 1];
     AttnParams p;
     p.q = (const __nv_bfloat16 *)q; p.k_cache = (const __nv_bfloat16 *)k_cache; p.v_cache = (const __nv_bfloat16 *)v_cache;
     p.out = (__nv_bfloat16 *)out; p.block_table = block_table; p.positions = positions;
     p.tile_seq = tile_seq; p.tile_t0 = tile_t0; p.tile_nt = tile_nt;
     p.part_o = (float *)scratch; p.part_ml = splits > 1 ? (float *)scratch + (size_t)T * H * splits * d : nullptr;
-    p.max_blocks = max_blocks; p.block_size = block_size; p.window = window; p.H = H; p.G = G; p.splits = splits;
+    p.max_blocks = max_blocks; p.block_size = block_size; p.window = window; p.H = H; p.G = G; p.kv_share = share; p.splits = splits;
     p.num_pages = num_pages; p.scale_log2 = scale * 1.4426950408889634f;
     p.sinks = sinks; p.slopes = slopes; p.zero_sink = zero_sink;
     p.head_scales = head_scales; p.softcap = softcap > 0.f ? softcap : 0.f; p.scale = scale;

@@ -157,6 +157,8 @@ def attention_step_arrays(q_lens, heads_per_group: int):
     out = {}
     for h in heights:
         per = (16 * int(h)) // heads_per_group if h != "16" else 2 * (128 // heads_per_group)
+        if max_q == 1:
+            per = max(per, 1)           # (the decode kernel cuts a larger group of heads into several)
         if per < 1:
             continue
         if max_q == 1:

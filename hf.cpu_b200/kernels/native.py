@@ -243,10 +243,14 @@ class NativeBackend:
             if tiling is not None:
                 tile_seq, tile_t0, tile_nt, n_tiles = tiling
                 splits, stages = 1, 2
+                groups = G
+                if decode_tma:
+                    # (more heads on a key/value head than a tile has rows: several groups, see the kernel)
+                    groups = G * next(s for s in range(1, H // G + 1) if H // G <= 16 * s and (H // G) % s == 0)
                 if decode:
                     # about `decode_ctas_per_sm` CTAs per SM in all; with one per SM the deep pipeline fits
                     hint = getattr(ctx, "decode_split_hint", max(1, ((ctx.max_kv_len + 63) // 64) // 2))
-                    splits = max(1, min(self.decode_ctas_per_sm * self.sm_count // max(1, n_tiles * G), hint))
+                    splits = max(1, min(self.decode_ctas_per_sm * self.sm_count // max(1, n_tiles * groups), hint))
                     stages = self.decode_stages
                 else:
                     # short portions over a long context (the end of a prompt, a prompt behind a shared prefix): few
@@ -258,7 +262,7 @@ class NativeBackend:
                     # the keys and values come by TMA, a warp of their own keeps them coming; the CTA that stores a
                     # tile's last split merges the splits (merge_in_kernel off: a second kernel does)
                     counters = None
-                    if self.merge_in_kernel and splits > 1 and n_tiles * G <= 4096:
+                    if self.merge_in_kernel and splits > 1 and n_tiles * groups <= 4096:
                         if self._counters is None or self._counters.device != q.device:
                             self._counters = torch.zeros(4096, dtype=torch.int32, device=q.device)
                         counters = self._counters
