@@ -136,6 +136,7 @@ latent_query_rope_kernel(const float *src, int splits, const float *cos_sin, int
         for (int s = 0; s < splits; s++) acc += p[(size_t)s * plane + c];
         qp[c] = from_f32<TO>(acc);
     }
+    if (rot == 0) return;
     int pos = positions[t];
     if (pos < 0 || pos >= n_positions) { if (lane == 0) atomicOr(err, HFB_ERR_POSITION); pos = 0; }
     const float *cs = cos_sin + (size_t)pos * (rot / 2) * 2;

@@ -74,6 +74,7 @@ class NativeBackend:
         self._counters = None
         self.branches = os.environ.get("HFB_BRANCHES", "1") != "0"        # independent work of a captured step as branches of the graph
         self._side = None
+        self.overlap = True                       # what set_launch_overlap was told last
         self.lib.hfb_linear_tc_partials_workspace.restype = ctypes.c_size_t
         self.lib.hfb_argmax2_scratch.restype = ctypes.c_size_t
         self.lib.hfb_decay_chunks_scratch.restype = ctypes.c_size_t
@@ -165,7 +166,8 @@ class NativeBackend:
                                                self._stream()), "rope_kv_write")
 
     def run_beside(self, first, second):
-        if not self.branches or not torch.cuda.is_current_stream_capturing():
+        # (launches that overlap with the kernel in front of them stay in one line)
+        if not self.branches or self.overlap or not torch.cuda.is_current_stream_capturing():
             first()
             second()
             return
@@ -179,6 +181,7 @@ class NativeBackend:
         here.wait_stream(self._side)
 
     def set_launch_overlap(self, on):
+        self.overlap = bool(on)
         self.lib.hfb_set_launch_overlap(c_int(1 if on else 0))
 
     def paged_attention(self, q, k_cache, v_cache, meta, ctx, H, G, d, window, scale, out, tile_arrays, dv=None, sinks=None,

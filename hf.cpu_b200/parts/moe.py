@@ -190,10 +190,16 @@ class MoeFfn(FeedForward):
         product and its partial sums are all summed by the norm's own pass."""
         if self.identity:
             raise UnsupportedError("identity experts are not summed by a norm's pass")
-        mix = self._experts(ctx, xn)
         if not self.FS:
-            return post.add_into(None, residual, next_norm, out, mix=mix)
-        hs = self._shared_hidden(ctx, xn)
+            return post.add_into(None, residual, next_norm, out, mix=self._experts(ctx, xn))
+        if self.gated:
+            # the shared expert's front product (never split, so it needs no scratch of the other's) beside the router, the
+            # grouping and the routed experts: two branches of a captured step
+            got = {}
+            kernels.run_beside(lambda: got.update(mix=self._experts(ctx, xn)), lambda: got.update(hs=self._shared_hidden(ctx, xn)))
+            mix, hs = got["mix"], got["hs"]
+        else:
+            mix, hs = self._experts(ctx, xn), self._shared_hidden(ctx, xn)
         with kernels.phase("down"):
             return post.add_product_into(hs, self.ws_down, None, y_buf, residual, next_norm, out, mix=mix)
 

@@ -92,7 +92,8 @@ def make_folder(cfg_dict, folder, seed, dtype=torch.float32, edit=None, sharp=2.
         elif name.endswith(".sink"):
             tensors[name] = uni(t, -2.0, 2.0)
         elif name.endswith(".correction"):
-            tensors[name] = uni(t, -0.7, 0.1)              # (most choice scores near or below zero)
+            # most choice scores near or below zero; stored in bfloat16 they lie far enough apart that few tokens are close calls
+            tensors[name] = -0.3 * torch.randperm(t.shape[0], generator=g).float() + uni(t, 0.0, 0.2) if soft else uni(t, -0.7, 0.1)
         elif name.endswith("loop.step"):
             tensors[name] = t * 0.7
         elif name == "embed":

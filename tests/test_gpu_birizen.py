@@ -361,11 +361,12 @@ FAMILIES = {"whole": traces.whole, "tail": traces.tail_one_by_one, "portions": t
 
 def assert_rows(got, ref, dtype, tol, what="the plain implementation"):
     """Every row within ``tol``; in bfloat16 some rows rest on a close call of a router (a choice between two nearly equal
-    scores flips with the rounding of its input, and later tokens read what this one left): up to 15 %, and never far off."""
+    scores flips with the rounding of its input, and later tokens read what this one left): up to 6 %; half of all rows are
+    well inside."""
     keys = sorted(got, key=lambda k: (str(k[0]), k[1]))
     errs = [float((got[k].double() - ref[k[0]][k[1]].double()).abs().max() / ref[k[0]][k[1]].double().abs().max()) for k in keys]
     over = [(k, e) for k, e in zip(keys, errs) if e > tol]
-    allowed = 0 if dtype == "float32" else max(1, int(0.15 * len(keys)))
+    allowed = 0 if dtype == "float32" else max(1, int(0.06 * len(keys)))
     assert len(over) <= allowed, (f"{len(over)} of {len(keys)} rows differ from {what}; first: request {over[0][0][0]} position "
                                   f"{over[0][0][1]} (error {over[0][1]:.3g})")
     if dtype == "bfloat16":
@@ -472,9 +473,44 @@ def test_greedy_generation_through_the_entry_point(folders):
         assert sess.engine.cache.pages_in_use() == 0
 
 
+@pytest.mark.parametrize("heads", [17, 20, 32, 40])
+@pytest.mark.parametrize("lens", [[300], [5, 130, 64]])
+def test_single_tokens_with_many_heads_on_one_latent_row(heads, lens):
+    """More query heads than the decode kernel's tiles have rows read the one cached row per token: against float64, with
+    sinks, one request with its keys split over blocks and several of unequal length."""
+    from hfcpu_b200.kernels import attention_step_arrays
+    d, bs, scale, dt, r = 128, 16, 0.12, torch.bfloat16, rng(heads)
+    pages_each = [(n + bs - 1) // bs for n in lens]
+    perm = np.random.default_rng(3).permutation(sum(pages_each) + 2)
+    kc = torch.zeros(len(perm), bs, 1, d, dtype=dt, device=DEV)
+    table = np.full((len(lens), max(pages_each)), -1)
+    keys, at = [], 0
+    for i, n in enumerate(lens):
+        k = dev(r.standard_normal((n, d)), dt)
+        keys.append(f64(k))
+        for j in range(pages_each[i]):
+            table[i, j] = perm[at]
+            part = k[j * bs:(j + 1) * bs]
+            kc[int(perm[at]), :part.shape[0], 0] = part
+            at += 1
+    from hfcpu_b200.engine.step import Workspace
+    ctx = SimpleNamespace(token_seq=i32(np.arange(len(lens))), positions=i32([n - 1 for n in lens]), max_q_len=1, max_kv_len=max(lens),
+                          buf=Workspace(torch.device(DEV)).get)
+    meta = SimpleNamespace(block_table=i32(table), block_size=bs, max_blocks=table.shape[1], group=0)
+    q, sinks = dev(r.standard_normal((len(lens), heads * d)), dt), dev(r.uniform(-2, 4, heads))
+    out = torch.full((len(lens), heads * d), float("nan"), dtype=dt, device=DEV)
+    K().paged_attention(q, kc, kc, meta, ctx, heads, 1, d, 0, scale, out, sinks=sinks,
+                        tiles={n: i32(a) for n, a in attention_step_arrays([1] * len(lens), heads).items()})
+    for i, k in enumerate(keys):
+        s = f64(q)[i].reshape(heads, d) @ k.T * scale
+        p = np.stack([plain.softmax_with_sink(s[h:h + 1], f64(sinks)[h])[0] for h in range(heads)])
+        assert rel(out[i].view(heads, d), p @ k) < 1.5e-2
+    K().check_device_errors()
+
+
 def test_bfloat16_generation_replays_graphs(folders):
-    """Steady decoding in bfloat16 goes through captured graphs (states, caches and passes included) and repeats itself; more
-    requests than slots, so that slots are used again."""
+    """Steady decoding in bfloat16 goes through captured graphs (states, caches and passes included; routed experts and shared
+    expert on two branches) and repeats itself; more requests than slots, so that slots are used again."""
     import hfcpu_b200
     sess = hfcpu_b200.Session(folders["wide16"], dtype="bfloat16", kv_block=16, kv_pages=128, max_seqs=2, ctx_max=512)
     prompts = list(requests(1032, [19, 130, 64, 5], seed=2).values())
