@@ -92,8 +92,9 @@ def make_folder(cfg_dict, folder, seed, dtype=torch.float32, edit=None, sharp=2.
         elif name.endswith(".sink"):
             tensors[name] = uni(t, -2.0, 2.0)
         elif name.endswith(".correction"):
-            # most choice scores near or below zero; stored in bfloat16 they lie far enough apart that few tokens are close calls
-            tensors[name] = -0.3 * torch.randperm(t.shape[0], generator=g).float() + uni(t, 0.0, 0.2) if soft else uni(t, -0.7, 0.1)
+            # most choice scores near or below zero; stored in bfloat16 they lie so far apart that close calls are rare (a choice
+            # that flips with rounding changes a row, and all later rows through the states, by more than rounding does)
+            tensors[name] = -0.25 * torch.randperm(t.shape[0], generator=g).float() + uni(t, 0.0, 0.02) if soft else uni(t, -0.7, 0.1)
         elif name.endswith("loop.step"):
             tensors[name] = t * 0.7
         elif name == "embed":
@@ -101,7 +102,7 @@ def make_folder(cfg_dict, folder, seed, dtype=torch.float32, edit=None, sharp=2.
         else:
             gain = 1.0
             if name.endswith(".router"):
-                gain = 1.5
+                gain = 0.35 if soft else 1.5
             elif name.endswith(".uq"):
                 gain = 1.0 if soft else sharp
             tensors[name] = t * gain / t.shape[1] ** 0.5
