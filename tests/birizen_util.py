@@ -68,8 +68,13 @@ FLAT = model(64, 48, 1e-5, [
     layer(latent(2, 16, 8, 16, 24, 24, 0.5, 50.0, (2.0, 32, 4.0, 1.0)), None),
     layer(lightning(16, 16, (0.95, 0.999)), moe(4, 2, 32, 1.0, (2, 1), (32, 1.0))),
 ])
-CONFIGS = {"odd": ODD, "wide": WIDE, "thin": THIN, "flat": FLAT}
-BLOCKS = {"odd": 8, "wide": 16, "thin": 4, "flat": 8}
+# Latent attention only (no state at all; launches may overlap), with a loop around the last of two layers.
+LATENT = model(130, 128, 1e-6, [
+    layer(latent(4, 32, 16, 32, 48, 48, 0.3, 1000.0, (4.0, 64, 8.0, 2.0)), moe(8, 3, 32, 1.0, (4, 2), (64, 1.5))),
+    layer(latent(2, 24, 8, 40, 32, 32, 0.4, 200.0), moe(4, 2, 40, 0.8, None, (48, 0.8))),
+], (1, 2, 2))
+CONFIGS = {"odd": ODD, "wide": WIDE, "thin": THIN, "flat": FLAT, "latent": LATENT}
+BLOCKS = {"odd": 8, "wide": 16, "thin": 4, "flat": 8, "latent": 8}
 
 
 def make_folder(cfg_dict, folder, seed, dtype=torch.float32, edit=None, sharp=2.5):

@@ -137,7 +137,7 @@ def test_every_pass_has_a_state_and_a_cache_of_its_own(folders, emu):
     assert eng.slots.entry_state(1) is None
 
 
-LENGTHS = {"odd": [1, 19, 70, 27], "wide": [3, 70, 20], "thin": [2, 9, 41], "flat": [17, 2, 33]}
+LENGTHS = {"odd": [1, 19, 70, 27], "wide": [3, 70, 20], "thin": [2, 9, 41], "flat": [17, 2, 33], "latent": [30, 2, 11]}
 
 
 @pytest.mark.parametrize("family", ["whole", "portions", "mixed"])

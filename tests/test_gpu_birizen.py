@@ -355,7 +355,7 @@ def folders(tmp_path_factory):
     return out
 
 
-LENGTHS = {"odd": [1, 19, 70, 130, 33], "wide": [3, 150, 64, 129, 220], "thin": [2, 9, 41], "flat": [65, 17, 2]}
+LENGTHS = {"odd": [1, 19, 70, 130, 33], "wide": [3, 150, 64, 129, 220], "thin": [2, 9, 41], "flat": [65, 17, 2], "latent": [70, 3, 33, 1]}
 FAMILIES = {"whole": traces.whole, "tail": traces.tail_one_by_one, "portions": traces.portions, "mixed": traces.mixed}
 
 
@@ -412,7 +412,7 @@ def test_cuttings_match_plain(folders, name, dtype, family):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("name", ["odd", "wide"])
+@pytest.mark.parametrize("name", ["odd", "wide", "latent"])
 def test_long_decoding(folders, name, dtype):
     """Every token a step of its own (from the second bfloat16 step on a replayed graph), two requests side by side, past
     several pages."""
